@@ -231,12 +231,16 @@ QS_API int qs_hyb_rope_append(void* proj, int64_t stride, const int32_t* tok_slo
 /* Optional parts of qs_hyb_attention / qs_hyb_attention_fast (a NULL pointer: none of them).
  * keep_first: with a window (and no chunks), positions < keep_first of the sequence stay visible to every later query.
  * slopes (fp32 [heads], may be NULL): slopes[h] * (query position - key position) is taken off head h's scaled score.
- * gate (storage type, may be NULL): head h's output of token t is multiplied by sigmoid(gate[t * gate_stride + h]). */
+ * gate (storage type, may be NULL): head h's output of token t is multiplied by sigmoid(gate[t * gate_stride + h]), or, with gate_wide, its
+ * output number j by sigmoid(gate[t * gate_stride + h * vdim + j]).
+ * softcap > 0: a scaled score s becomes softcap * tanh(s / softcap), ahead of the slopes and the mask (needs scale > 0). */
 typedef struct {
   int keep_first;
   const float* slopes;
   const void* gate;
   int64_t gate_stride;
+  int gate_wide;
+  float softcap;
 } qs_attn_extra;
 /* causal attention of every token over positions first..tok_pos of its sequence in the paged cache, `maps` (1 or 2) softmax maps per head
  * over shared values: o = a1 [- lambda a2]; head_norm: o *= rsqrt(mean(o^2) + eps); o *= out_scale.  out [tokens, heads*vdim].
@@ -290,12 +294,13 @@ QS_API int qs_hyb_branch_norm_mean(float* y, const void* a, const void* b, const
  * entries (rot_layout 0: pairs (2i, 2i+1); 1: pairs (i, i + rot_dims/2); angle = position * inv_freq[i]; rot_dims 0: none); queries times
  * q_factor[head], in place.  Keys and values (+ bias) go to the pages K [page][page_size][G][dim], V [page][page_size][G][vdim].
  * q_gain / k_gain (fp32 [dim], may be NULL): gains of the unit-RMS heads, shared by the heads.  tied_values: the rows have no v part, a key
- * head's value is that key head as projected (+ bias), not yet normed (vdim == dim). */
+ * head's value is that key head as projected (+ bias), not yet normed (vdim == dim).  value_rms: value heads (+ bias) are stored at
+ * unit RMS, v *= rsqrt(mean(v^2) + eps). */
 QS_API int qs_hyb_qk_prepare_append(void* proj, int64_t stride, const float* bias, const float* q_factor, const int32_t* tok_slot,
                                     const int32_t* tok_pos, const int32_t* block_table, int max_blocks, void* kpool, void* vpool,
                                     const float* inv_freq, int rot_layout, int rot_dims, int unit_rms, float eps, int tokens_n, int heads,
                                     int kv_heads, int dim, int vdim, int page_size, const float* q_gain, const float* k_gain, int tied_values,
-                                    int dtype, void* stream);
+                                    int value_rms, int dtype, void* stream);
 /* Gate recurrence (HGRN2) over projection rows [H*dim q | H*dim f | H*vdim v]: q <- silu(q), f <- lower + (1 - lower) sigmoid(f + f_bias)
  * (fp32 [H*dim] each), per head S <- diag(f) S + (1 - f) v^T, o = S^T q, out = o rsqrt(mean(o^2) + eps) norm_w (fp32 [vdim], may be NULL).
  * state fp32 [slots, H, dim, vdim]; a run that starts at position 0 starts from zero.  prep fp32 [tokens, 2 H dim + H vdim] and o_raw fp32
@@ -361,6 +366,13 @@ QS_API int qs_hyb_bias_gelu_tanh(void* out, int64_t out_stride, const void* in, 
  * [width], may be NULL); out_h (may be NULL) <- x in the storage type.  add rows: fp32 if add_f32, else storage type; x fp32 [tokens, width]. */
 QS_API int qs_hyb_post_norm_update(void* out_h, float* x, const void* add, int add_f32, const float* add_bias, const float* w, const float* ls,
                                    float offset, float eps, int tokens_n, int width, int dtype, void* stream);
+/* Residual update of blocks that norm a sublayer's input and its output, with a gate per channel on the output: y = add (+ add_bias, fp32
+ * [width], may be NULL); (gate != NULL) y *= sigmoid(gate[t * gate_stride + i] + gate_bias[i]) (gate storage type, gate_bias fp32, may be
+ * NULL); x <- (fresh ? 0 : x) + mult gnorm(y) (offset + w); (out_h != NULL) out_h <- gnorm(x) (offset + w_next), storage type.  gnorm:
+ * y_i rsqrt(m + eps), m the mean square of the width / groups neighbouring columns of i's group.  add rows: fp32 if add_f32, else storage type. */
+QS_API int qs_hyb_gated_norm_update(void* out_h, float* x, int fresh, const void* add, int add_f32, const float* add_bias, const void* gate,
+                                    int64_t gate_stride, const float* gate_bias, const float* w, float mult, const float* w_next, int groups,
+                                    float offset, float eps, int tokens_n, int width, int dtype, void* stream);
 /* out[i] = x[i] in the storage type (x fp32) */
 QS_API int qs_hyb_cast_rows(void* out, const float* x, int64_t n, int dtype, void* stream);
 /* out[t, i] = act(in[t, i] + bias[i]) * (in[t, ff + i] + bias[ff + i]) (bias fp32 [2 ff], may be NULL); rows of in_stride / out_stride elements */

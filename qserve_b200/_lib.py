@@ -65,9 +65,10 @@ SIGNATURES = {
     # csrc/hybrid_blocks.cu, csrc/hybrid_linear.cu
     "qs_hyb_stream_norm": (c_int, [_P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _I, _F, _F, _I, _I, _I, _P]),
     "qs_hyb_branch_norm_mean": (c_int, [_P, _P, _P, _P, _P, _F, _F, _I, _I, _I, _P]),
-    "qs_hyb_qk_prepare_append": (c_int, [_P, _L, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P]),
+    "qs_hyb_qk_prepare_append": (c_int, [_P, _L, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P]),
     "qs_hyb_gated_linear": (c_int, [_P, _L, _P, _P, _P, _L, _P, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P]),
     "qs_hyb_post_norm_update": (c_int, [_P, _P, _P, _I, _P, _P, _P, _F, _F, _I, _I, _I, _P]),
+    "qs_hyb_gated_norm_update": (c_int, [_P, _P, _I, _P, _I, _P, _P, _L, _P, _P, _F, _P, _I, _F, _F, _I, _I, _I, _P]),
     "qs_hyb_cast_rows": (c_int, [_P, _P, _L, _I, _P]),
     "qs_hyb_bias_gated_act": (c_int, [_P, _L, _P, _L, _P, _I, _I, _I, _I, _P]),
     "qs_hyb_gate_recurrence": (c_int, [_P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P]),
@@ -96,8 +97,9 @@ ABI_VERSION = 1
 
 
 class AttnExtra(ctypes.Structure):
-    """qs_attn_extra: optional parts of the attention kernels (kept first positions of a window, distance-bias slopes, a sigmoid gate per head)."""
-    _fields_ = [("keep_first", c_int), ("slopes", c_void_p), ("gate", c_void_p), ("gate_stride", c_int64)]
+    """qs_attn_extra: optional parts of the attention kernels (kept first positions of a window, distance-bias slopes, a sigmoid gate per head or
+    per output number, a tanh cap on the scores)."""
+    _fields_ = [("keep_first", c_int), ("slopes", c_void_p), ("gate", c_void_p), ("gate_stride", c_int64), ("gate_wide", c_int), ("softcap", c_float)]
 
 
 def _load() -> ctypes.CDLL:

@@ -253,7 +253,9 @@ __global__ void __launch_bounds__(kAttnThreads) paged_multimap_attention_kernel(
         float d = 0.f;
         for (int i = lane; i < D; i += 32) d += qs[m * D + i] * ldf(kr + m * D + i);
         d = warp_sum(d);
-        if (lane == 0) ps[m * kAttnKT + j] = d * scale - slope * (float)(pos - kj);
+        d *= scale;
+        if (ex.softcap > 0.f) d = ex.softcap * tanhf(d / ex.softcap);
+        if (lane == 0) ps[m * kAttnKT + j] = d - slope * (float)(pos - kj);
       }
     }
     __syncthreads();
@@ -315,12 +317,16 @@ __global__ void __launch_bounds__(kAttnThreads) paged_multimap_attention_kernel(
     ss = block_sum(ss, red);
     r *= 1.f / sqrtf(ss / (float)Dv + eps);
   }
-  if (ex.gate != nullptr) r *= sigmoid_f(ldf(static_cast<const ST*>(ex.gate) + (size_t)t * ex.gate_stride + h));
+  const ST* gate = static_cast<const ST*>(ex.gate) + (ex.gate != nullptr ? (size_t)t * ex.gate_stride : 0);
+  if (ex.gate != nullptr && !ex.gate_wide) r *= sigmoid_f(ldf(gate + h));
   ST* orow = out + (size_t)t * out_stride + (size_t)h * Dv;
 #pragma unroll
   for (int j = 0; j < kAttnMaxV; ++j) {
     const int d = threadIdx.x + j * kAttnThreads;
-    if (d < Dv) stf(orow + d, o[j] * r);
+    if (d >= Dv) continue;
+    float v = o[j] * r;
+    if (ex.gate != nullptr && ex.gate_wide) v *= sigmoid_f(ldf(gate + (size_t)h * Dv + d));
+    stf(orow + d, v);
   }
 }
 
@@ -339,7 +345,7 @@ __global__ void __launch_bounds__(128, KT == 32 ? 3 : 2) tile_attention_kernel(
     const __nv_bfloat16* __restrict__ vpool, const int* __restrict__ tile_entry, const int* __restrict__ tile_row0,
     const int* __restrict__ entry_start, const int* __restrict__ entry_len, const int* __restrict__ entry_slot, const int* __restrict__ entry_pos0,
     const int* __restrict__ block_table, int max_blocks, int H, int G, int maps, int D, float scale, int page, int chunk, int window,
-    const float* __restrict__ sinks, int keep, const float* __restrict__ slopes) {
+    const float* __restrict__ sinks, int keep, const float* __restrict__ slopes, float cap_in, float cap_out) {
   extern __shared__ __align__(16) unsigned char smraw[];
   constexpr int Dv = NVT * 16;
   const int SD = D + kPad, SV = Dv + kPad;
@@ -368,7 +374,8 @@ __global__ void __launch_bounds__(128, KT == 32 ? 3 : 2) tile_attention_kernel(
   const int n_pre = kept_tiles(first_key(qpos0, chunk, window), keep, KT), n_walk = n_pre + n_kt - kt_lo;  // kept first positions, then the rest
   auto tile_at = [&](int i) { return i < n_pre ? i : kt_lo + i - n_pre; };
   const float slope2 = slopes != nullptr ? slopes[h] * 1.4426950408889634f : 0.f;
-  const float scale_log2 = scale * 1.4426950408889634f;
+  // capped scores (cap_in = scale / cap, cap_out = cap in the base-2 domain) leave cap_scores as they enter the softmax
+  const float scale_log2 = cap_in > 0.f ? 1.f : scale * 1.4426950408889634f;
   const int qrow = warp * 16 + (lane >> 2);  // this thread's rows: qrow, qrow + 8
   const int fk[2] = {first_key(qpos0 + qrow, chunk, window), first_key(qpos0 + qrow + 8, chunk, window)};
   const int warp_fk = first_key(min(last_qpos, qpos0 + warp * 16 + 15), chunk, window);  // the largest first key among the warp's rows
@@ -429,6 +436,7 @@ __global__ void __launch_bounds__(128, KT == 32 ? 3 : 2) tile_attention_kernel(
         mma_bf16(s[2 * np + 1], a, b[2], b[3]);
       }
     }
+    if (cap_in > 0.f) cap_scores(s, cap_in, cap_out);
     // scale, causal mask, online softmax (rows qrow and qrow + 8; a row's columns live in the 4 lanes of a quad)
     float mx[2] = {-INFINITY, -INFINITY};
     const bool diagonal = kt * KT + KT - 1 > qpos0 + warp * 16 || kt * KT < warp_fk;
@@ -521,7 +529,7 @@ __global__ void __launch_bounds__(128, KT == 32 ? 3 : 2) tile_attention_kernel(
 template <typename ST>
 __global__ void multimap_combine_kernel(ST* __restrict__ out, long long out_stride, const float* __restrict__ a_in, const int* __restrict__ tok_list,
                                         int n_list, int H, int maps, int Dv, float lambda, float out_scale, float eps, int head_norm,
-                                        const ST* __restrict__ gate, long long gate_stride) {
+                                        const ST* __restrict__ gate, long long gate_stride, int gate_wide) {
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (w >= n_list * H) return;
   const int t = tok_list[w / H], h = w % H;
@@ -533,8 +541,13 @@ __global__ void multimap_combine_kernel(ST* __restrict__ out, long long out_stri
   }
   ss = warp_sum(ss);
   float r = head_norm ? out_scale / sqrtf(ss / (float)Dv + eps) : out_scale;
-  if (gate != nullptr) r *= sigmoid_f(ldf(gate + (size_t)t * gate_stride + h));
+  if (gate != nullptr && !gate_wide) r *= sigmoid_f(ldf(gate + (size_t)t * gate_stride + h));
   ST* dst = out + (size_t)t * out_stride + (size_t)h * Dv;
+  if (gate != nullptr && gate_wide) {
+    const ST* gr = gate + (size_t)t * gate_stride + (size_t)h * Dv;
+    for (int i = lane; i < Dv; i += 32) stf(dst + i, (maps == 2 ? a[i] - lambda * a[Dv + i] : a[i]) * r * fast_sigmoid(ldf(gr + i)));
+    return;
+  }
   for (int i = lane; i < Dv; i += 32) stf(dst + i, (maps == 2 ? a[i] - lambda * a[Dv + i] : a[i]) * r);
 }
 
@@ -551,7 +564,7 @@ __global__ void __launch_bounds__(128) group_attention_kernel(
     float* __restrict__ part, const __nv_bfloat16* __restrict__ q, long long q_stride, const __nv_bfloat16* __restrict__ kpool,
     const __nv_bfloat16* __restrict__ vpool, const int* __restrict__ tok_list, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     const int* __restrict__ block_table, int max_blocks, int H, int G, int maps, int D, float scale, int page, int shares, int chunk, int window,
-    int keep, const float* __restrict__ slopes) {
+    int keep, const float* __restrict__ slopes, float cap_in, float cap_out) {
   extern __shared__ __align__(16) unsigned char smraw[];
   constexpr int Dv = NVT * 16;
   const int SD = D + kPad, SV = Dv + kPad, R = H / G;
@@ -584,7 +597,7 @@ __global__ void __launch_bounds__(128) group_attention_kernel(
 #pragma unroll
   for (int i = 0; i < 2 * NVT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const float scale_log2 = cap_in > 0.f ? 1.f : scale * 1.4426950408889634f;  // capped scores leave cap_scores as they enter the softmax
   // two threads per key row, alternating 16-byte chunks: one block-table lookup per thread and tile, made one tile ahead of its use so
   // that the lookup's latency hides behind a tile of arithmetic
   auto cell_of = [&](int kt) -> long long {
@@ -638,6 +651,7 @@ __global__ void __launch_bounds__(128) group_attention_kernel(
       mma_bf16(s[0], a, b[0], b[1]);
       mma_bf16(s[1], a, b[2], b[3]);
     }
+    if (cap_in > 0.f) cap_scores(s, cap_in, cap_out);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -738,7 +752,7 @@ __global__ void __launch_bounds__(128) group_attention_kernel(
 template <typename ST>
 __global__ void group_merge_kernel(ST* __restrict__ out, long long out_stride, const float* __restrict__ part, const int* __restrict__ tok_list,
                                    int n_list, int H, int maps, int Dv, int shares, float lambda, float out_scale, float eps, int head_norm,
-                                   const float* __restrict__ sinks, const ST* __restrict__ gate, long long gate_stride) {
+                                   const float* __restrict__ sinks, const ST* __restrict__ gate, long long gate_stride, int gate_wide) {
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (w >= n_list * H) return;
   const int li = w / H, h = w - li * H, t = tok_list[li];
@@ -772,11 +786,12 @@ __global__ void group_merge_kernel(ST* __restrict__ out, long long out_stride, c
   for (int j = 0; j < 8; ++j) ss += ov[j] * ov[j];
   ss = warp_sum(ss);
   float r = head_norm ? out_scale / sqrtf(ss / (float)Dv + eps) : out_scale;
-  if (gate != nullptr) r *= sigmoid_f(ldf(gate + (size_t)t * gate_stride + h));
+  const ST* gr = gate != nullptr ? gate + (size_t)t * gate_stride + (gate_wide ? (size_t)h * Dv : (size_t)h) : nullptr;
+  if (gate != nullptr && !gate_wide) r *= sigmoid_f(ldf(gr));
   ST* dst = out + (size_t)t * out_stride + (size_t)h * Dv;
 #pragma unroll
   for (int j = 0; j < 8; ++j)
-    if (lane + 32 * j < Dv) stf(dst + lane + 32 * j, ov[j] * r);
+    if (lane + 32 * j < Dv) stf(dst + lane + 32 * j, ov[j] * r * (gate != nullptr && gate_wide ? fast_sigmoid(ldf(gr + lane + 32 * j)) : 1.f));
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------------
@@ -1047,8 +1062,12 @@ __global__ void delta_gate_out_kernel(ST* __restrict__ out, long long out_stride
 }
 
 inline AttnExtra attn_extra(const qs_attn_extra* e) {
-  return e != nullptr ? AttnExtra{e->keep_first, e->slopes, e->gate, (long long)e->gate_stride} : AttnExtra{0, nullptr, nullptr, 0};
+  return e != nullptr ? AttnExtra{e->keep_first, e->slopes, e->gate, (long long)e->gate_stride, e->gate_wide, e->softcap}
+                      : AttnExtra{0, nullptr, nullptr, 0, 0, 0.f};
 }
+// the two factors of a capped score on the tensor-core kernels: tanh's argument per unit of q . k, and the cap in the base-2 domain
+inline float cap_in(const AttnExtra& ex, float scale) { return ex.softcap > 0.f ? scale / ex.softcap : 0.f; }
+inline float cap_out(const AttnExtra& ex) { return ex.softcap * 1.4426950408889634f; }
 
 template <typename ST>
 int launch_attention(void* out, long long out_stride, const void* q, long long q_stride, const void* kpool, const void* vpool, const int* tok_slot,
@@ -1094,7 +1113,7 @@ int launch_tiles(float* scratch, const void* q, long long q_stride, const void* 
   }
   tile_attention_kernel<NVT, 3, KT><<<dim3(n_tiles, H * maps), 128, smem, s>>>(scratch, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)kpool,
       (const __nv_bfloat16*)vpool, tile_entry, tile_row0, entry_start, entry_len, entry_slot, entry_pos0, block_table, max_blocks, H, G, maps, D, scale, page, chunk, window, sinks,
-      ex.keep_first, ex.slopes);
+      ex.keep_first, ex.slopes, cap_in(ex, scale), cap_out(ex));
   return check_cuda(cudaGetLastError(), "hyb_attention tiles");
 }
 
@@ -1119,11 +1138,11 @@ int launch_group(void* out, long long out_stride, float* part, const void* q, lo
   const int shares = group_shares(n_list, G, maps);
   group_attention_kernel<NVT, 3><<<dim3(n_list, G * maps, shares), 128, smem, s>>>(part, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)kpool,
       (const __nv_bfloat16*)vpool, tok_list, tok_slot, tok_pos, block_table, max_blocks, H, G, maps, D, scale, page, shares, chunk, window, ex.keep_first,
-      ex.slopes);
+      ex.slopes, cap_in(ex, scale), cap_out(ex));
   const int warps = n_list * H;
   group_merge_kernel<__nv_bfloat16><<<(warps + 3) / 4, 128, 0, s>>>((__nv_bfloat16*)out, out_stride, part, tok_list, n_list, H, maps, NVT * 16, shares,
                                                                      lambda, out_scale, eps, head_norm, sinks, (const __nv_bfloat16*)ex.gate,
-                                                                     ex.gate_stride);
+                                                                     ex.gate_stride, ex.gate_wide);
   return check_cuda(cudaGetLastError(), "hyb_attention single tokens");
 }
 
@@ -1261,6 +1280,7 @@ int qs_hyb_attention(void* out, int64_t out_stride, const void* q, int64_t q_str
   QS_REQUIRE(out && q && kpool && vpool && tok_slot && tok_pos && block_table, "hyb_attention: null tensor");
   QS_REQUIRE(chunk >= 0 && window >= 0, "hyb_attention: negative chunk or window");
   const AttnExtra ex = attn_extra(extra);
+  QS_REQUIRE(ex.softcap >= 0.f && (ex.softcap == 0.f || scale > 0.f), "hyb_attention: a score cap is positive and goes with a positive scale");
   QS_REQUIRE(ex.keep_first >= 0 && (ex.keep_first == 0 || (window > 0 && chunk == 0)), "hyb_attention: kept first positions go with a window and no chunks");
   QS_REQUIRE(maps == 1 || maps == 2, "hyb_attention: 1 or 2 softmax maps per head");
   QS_REQUIRE(heads % kv_heads == 0 && vdim <= kAttnThreads * kAttnMaxV && page_size > 0, "hyb_attention: bad head geometry (vdim <= 512)");
@@ -1293,6 +1313,7 @@ int qs_hyb_attention_fast(void* out, int64_t out_stride, const void* q, int64_t 
                           void* stream) {
   QS_REQUIRE(chunk >= 0 && window >= 0, "hyb_attention_fast: negative chunk or window");
   const AttnExtra ex = attn_extra(extra);
+  QS_REQUIRE(ex.softcap >= 0.f && (ex.softcap == 0.f || scale > 0.f), "hyb_attention_fast: a score cap is positive and goes with a positive scale");
   QS_REQUIRE(ex.keep_first >= 0 && (ex.keep_first == 0 || (window > 0 && chunk == 0)), "hyb_attention_fast: kept first positions go with a window and no chunks");
   QS_REQUIRE(out && q && kpool && vpool && tok_slot && tok_pos && block_table, "hyb_attention_fast: null tensor");
   QS_REQUIRE(fast_attention_supported(dtype, heads, kv_heads, maps, dim, vdim, q_stride), "hyb_attention_fast: shape not supported (use qs_hyb_attention)");
@@ -1315,7 +1336,8 @@ int qs_hyb_attention_fast(void* out, int64_t out_stride, const void* q, int64_t 
     if (rc) return rc;
     const int warps = n_long * heads;
     multimap_combine_kernel<__nv_bfloat16><<<(warps + 3) / 4, 128, 0, s>>>((__nv_bfloat16*)out, out_stride, scratch, long_tokens, n_long, heads, maps, vdim,
-                                                                          lambda, out_scale, eps, head_norm, (const __nv_bfloat16*)ex.gate, ex.gate_stride);
+                                                                          lambda, out_scale, eps, head_norm, (const __nv_bfloat16*)ex.gate, ex.gate_stride,
+                                                                          ex.gate_wide);
   }
   if (n_short > 0) {
     int rc = 0;

@@ -225,7 +225,7 @@ __global__ void branch_norm_mean_vec_kernel(float* __restrict__ y, const ST* __r
 //   projection row: [H*D q | G*D k | G*Dv v];  bias (fp32, same layout) may be null
 //   per head, in this order: + bias;  (unit_rms) x <- x * rsqrt(mean(x^2) + eps) [* q_gain or k_gain, fp32 [D] shared by the heads];  rotary
 //   on the first rot_dims entries (layout 0: pairs (2i, 2i+1), layout 1: pairs (i, i + rot_dims/2); angle = position * inv_freq[i]);  queries
-//   times q_factor[head] (may be null).  tied_values: the row has no v part, a key head's value is that key head as projected (+ bias), not yet normed.
+//   times q_factor[head] (may be null).  value_rms: value heads (+ bias) are brought to unit RMS over Dv before they are stored.  tied_values: the row has no v part, a key head's value is that key head as projected (+ bias), not yet normed.
 // grid (tokens, H + G): the first H blocks finish a query head in place, the others store a key head and its value head (+ bias) in the pages
 // K [page][page_size][G][D], V [page][page_size][G][Dv].
 // ---------------------------------------------------------------------------------------------------------------------------------
@@ -234,7 +234,7 @@ __global__ void qk_prepare_append_kernel(ST* __restrict__ proj, long long stride
                                          const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, const int* __restrict__ block_table,
                                          int max_blocks, ST* __restrict__ kpool, ST* __restrict__ vpool, const float* __restrict__ inv_freq,
                                          int rot_layout, int rot_dims, int unit_rms, float eps, int H, int G, int D, int Dv, int page,
-                                         const float* __restrict__ q_gain, const float* __restrict__ k_gain, int tied_values) {
+                                         const float* __restrict__ q_gain, const float* __restrict__ k_gain, int tied_values, int value_rms) {
   extern __shared__ float hs[];  // the head, D floats
   __shared__ float red[33];
   const int t = blockIdx.x, u = blockIdx.y;
@@ -264,11 +264,17 @@ __global__ void qk_prepare_append_kernel(ST* __restrict__ proj, long long stride
     dst = kpool + (cell * G + g) * (size_t)D;
     const size_t v0 = (size_t)(H + G) * D + (size_t)g * Dv;
     ST* vd = vpool + (cell * G + g) * (size_t)Dv;
-    if (tied_values) {
-      for (int i = threadIdx.x; i < D; i += blockDim.x) stf(vd + i, hs[i]);
-    } else {
-      for (int i = threadIdx.x; i < Dv; i += blockDim.x) stf(vd + i, ldf(row + v0 + i) + (bias != nullptr ? bias[v0 + i] : 0.f));
+    auto value = [&](int i) { return tied_values ? hs[i] : ldf(row + v0 + i) + (bias != nullptr ? bias[v0 + i] : 0.f); };
+    float rv = 1.f;
+    if (value_rms) {
+      float sv = 0.f;
+      for (int i = threadIdx.x; i < Dv; i += blockDim.x) {
+        const float v = value(i);
+        sv += v * v;
+      }
+      rv = 1.f / sqrtf(block_sum(sv, red) / (float)Dv + eps);
     }
+    for (int i = threadIdx.x; i < Dv; i += blockDim.x) stf(vd + i, value(i) * rv);
   }
   const float* gain = is_q ? q_gain : k_gain;
   if (gain != nullptr) {
@@ -793,6 +799,117 @@ __global__ void post_norm_update_kernel(ST* __restrict__ out_h, float* __restric
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------------------------------
+// Residual update of blocks that norm a sublayer's input and its output, with a gate per channel on the output:
+//   y = add [+ add_bias];  (gate != null) y <- y * sigmoid(gate + gate_bias);  x <- [x +] mult * gnorm(y) * (offset + w);
+//   (out_h != null) out_h <- gnorm(x) * (offset + w_next)                     (storage type: the next sublayer's input)
+// gnorm: y_i -> y_i rsqrt(m + eps), m the mean square of the W / groups neighbouring columns that make i's group.  fresh: x is not read (the row
+// starts the stream).  add: rows fp32 if add_f32, else of the storage type; gate: storage type, rows of gate_stride elements.
+// One block per token.  The vector kernel keeps the row in registers (one pass over memory): per = warps / groups warps share a group, a
+// thread holds NV chunks of four columns of one group; a group's sum is its warps' sums added in a fixed order.
+// ---------------------------------------------------------------------------------------------------------------------------------
+template <typename ST, int NV>
+__global__ void __launch_bounds__(512) gated_norm_update_vec_kernel(ST* __restrict__ out_h, float* __restrict__ x, int fresh, const void* __restrict__ add, int add_f32,
+                                             const float* __restrict__ add_bias, const ST* __restrict__ gate, long long gate_stride,
+                                             const float* __restrict__ gate_bias, const float* __restrict__ w, float mult, const float* __restrict__ w_next,
+                                             int groups, float offset, float eps, int W) {
+  __shared__ float red[2][32];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = (blockDim.x >> 5) / groups, g = warp / per, sub = warp - g * per, part = W / groups;
+  const size_t base = (size_t)blockIdx.x * W;
+  float4 y[NV], v[NV], z[NV];
+  bool live[NV];
+  int col[NV];
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {  // every load of the row is in flight before the first sum
+    const int c = ((sub + k * per) * 32 + lane) * 4;
+    live[k] = c < part;
+    col[k] = g * part + (live[k] ? c : 0);
+    const int i = col[k];
+    y[k] = add_f32 ? ld4(static_cast<const float*>(add) + base + i) : ld4(static_cast<const ST*>(add) + base + i);
+    v[k] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : ld4(x + base + i);
+    if (gate != nullptr) z[k] = ld4(gate + (size_t)blockIdx.x * gate_stride + i);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = col[k];
+    if (add_bias != nullptr) { const float4 b = ld4(add_bias + i); y[k].x += b.x; y[k].y += b.y; y[k].z += b.z; y[k].w += b.w; }
+    if (gate != nullptr) {
+      if (gate_bias != nullptr) { const float4 b = ld4(gate_bias + i); z[k].x += b.x; z[k].y += b.y; z[k].z += b.z; z[k].w += b.w; }
+      if (sizeof(ST) == 2) {
+        y[k].x *= fast_sigmoid(z[k].x); y[k].y *= fast_sigmoid(z[k].y); y[k].z *= fast_sigmoid(z[k].z); y[k].w *= fast_sigmoid(z[k].w);
+      } else {
+        y[k].x *= sigmoid_f(z[k].x); y[k].y *= sigmoid_f(z[k].y); y[k].z *= sigmoid_f(z[k].z); y[k].w *= sigmoid_f(z[k].w);
+      }
+    }
+    if (live[k]) ss += (y[k].x * y[k].x + y[k].y * y[k].y) + (y[k].z * y[k].z + y[k].w * y[k].w);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red[0][warp] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int j = 0; j < per; ++j) tot += red[0][g * per + j];
+  const float r = mult / sqrtf(tot / (float)part + eps);
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    if (!live[k]) continue;
+    const float4 a = ld4(w + col[k]);
+    v[k].x += y[k].x * r * (offset + a.x); v[k].y += y[k].y * r * (offset + a.y); v[k].z += y[k].z * r * (offset + a.z); v[k].w += y[k].w * r * (offset + a.w);
+    st4(x + base + col[k], v[k]);
+    ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+  }
+  if (out_h == nullptr) return;
+  ss = warp_sum(ss);
+  if (lane == 0) red[1][warp] = ss;
+  __syncthreads();
+  tot = 0.f;
+  for (int j = 0; j < per; ++j) tot += red[1][g * per + j];
+  const float q = 1.f / sqrtf(tot / (float)part + eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    if (!live[k]) continue;
+    const float4 a = ld4(w_next + col[k]);
+    st4(out_h + base + col[k], make_float4(v[k].x * q * (offset + a.x), v[k].y * q * (offset + a.y), v[k].z * q * (offset + a.z), v[k].w * q * (offset + a.w)));
+  }
+}
+
+// any width and number of groups: the row passes through shared memory, a warp sums a group
+template <typename ST>
+__global__ void gated_norm_update_kernel(ST* __restrict__ out_h, float* __restrict__ x, int fresh, const void* __restrict__ add, int add_f32,
+                                         const float* __restrict__ add_bias, const ST* __restrict__ gate, long long gate_stride,
+                                         const float* __restrict__ gate_bias, const float* __restrict__ w, float mult, const float* __restrict__ w_next,
+                                         int groups, float offset, float eps, int W) {
+  extern __shared__ float dyn[];  // the row [W] | 1 / rms [groups]
+  float* rinv = dyn + W;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, part = W / groups;
+  const size_t base = (size_t)blockIdx.x * W;
+  auto group_scales = [&](float factor) {
+    __syncthreads();
+    for (int g = warp; g < groups; g += nw) {
+      float ss = 0.f;
+      for (int i = lane; i < part; i += 32) ss += dyn[g * part + i] * dyn[g * part + i];
+      ss = warp_sum(ss);
+      if (lane == 0) rinv[g] = factor / sqrtf(ss / (float)part + eps);
+    }
+    __syncthreads();
+  };
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    float y = (add_f32 ? static_cast<const float*>(add)[base + i] : ldf(static_cast<const ST*>(add) + base + i)) + (add_bias != nullptr ? add_bias[i] : 0.f);
+    if (gate != nullptr) y *= sigmoid_f(ldf(gate + (size_t)blockIdx.x * gate_stride + i) + (gate_bias != nullptr ? gate_bias[i] : 0.f));
+    dyn[i] = y;
+  }
+  group_scales(mult);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = (fresh ? 0.f : x[base + i]) + dyn[i] * rinv[i / part] * (offset + w[i]);
+    x[base + i] = v;
+    dyn[i] = v;
+  }
+  if (out_h == nullptr) return;
+  group_scales(1.f);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) stf(out_h + base + i, dyn[i] * rinv[i / part] * (offset + w_next[i]));
+}
+
 // storage-type copy of fp32 rows (the input of a sublayer that takes the un-normed stream)
 template <typename ST>
 __global__ void cast_rows_kernel(ST* __restrict__ out, const float* __restrict__ x, size_t n) {
@@ -930,7 +1047,7 @@ int qs_hyb_branch_norm_mean(float* y, const void* a, const void* b, const float*
 int qs_hyb_qk_prepare_append(void* proj, int64_t stride, const float* bias, const float* q_factor, const int32_t* tok_slot, const int32_t* tok_pos,
                              const int32_t* block_table, int max_blocks, void* kpool, void* vpool, const float* inv_freq, int rot_layout,
                              int rot_dims, int unit_rms, float eps, int tokens_n, int heads, int kv_heads, int dim, int vdim, int page_size,
-                             const float* q_gain, const float* k_gain, int tied_values, int dtype, void* stream) {
+                             const float* q_gain, const float* k_gain, int tied_values, int value_rms, int dtype, void* stream) {
   QS_REQUIRE(proj && tok_slot && tok_pos && block_table && kpool && vpool, "hyb_qk_prepare_append: null tensor");
   QS_REQUIRE(!tied_values || vdim == dim, "hyb_qk_prepare_append: values tied to the keys need vdim == dim");
   QS_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || inv_freq != nullptr) && (rot_layout == 0 || rot_layout == 1),
@@ -944,10 +1061,10 @@ int qs_hyb_qk_prepare_append(void* proj, int64_t stride, const float* bias, cons
         (qk_prepare_append_kernel<__nv_bfloat16><<<grid, 64, smb, s>>>((__nv_bfloat16*)proj, stride, bias, q_factor, tok_slot, tok_pos, block_table,
                                                                         max_blocks, (__nv_bfloat16*)kpool, (__nv_bfloat16*)vpool, inv_freq, rot_layout,
                                                                         rot_dims, unit_rms, eps, heads, kv_heads, dim, vdim, page_size, q_gain, k_gain,
-                                                                        tied_values)),
+                                                                        tied_values, value_rms)),
         (qk_prepare_append_kernel<float><<<grid, 64, smb, s>>>((float*)proj, stride, bias, q_factor, tok_slot, tok_pos, block_table, max_blocks,
                                                                 (float*)kpool, (float*)vpool, inv_freq, rot_layout, rot_dims, unit_rms, eps, heads,
-                                                                kv_heads, dim, vdim, page_size, q_gain, k_gain, tied_values)));
+                                                                kv_heads, dim, vdim, page_size, q_gain, k_gain, tied_values, value_rms)));
   return check_cuda(cudaGetLastError(), "hyb_qk_prepare_append");
 }
 
@@ -1107,6 +1224,50 @@ int qs_hyb_post_norm_update(void* out_h, float* x, const void* add, int add_f32,
           (post_norm_update_kernel<float, false><<<tokens_n, threads, 0, s>>>((float*)out_h, x, add, add_f32, add_bias, w, ls, offset, eps, width)));
   }
   return check_cuda(cudaGetLastError(), "hyb_post_norm_update");
+}
+
+int qs_hyb_gated_norm_update(void* out_h, float* x, int fresh, const void* add, int add_f32, const float* add_bias, const void* gate, int64_t gate_stride,
+                             const float* gate_bias, const float* w, float mult, const float* w_next, int groups, float offset, float eps,
+                             int tokens_n, int width, int dtype, void* stream) {
+  QS_REQUIRE(x && add && w && (out_h == nullptr || w_next != nullptr), "hyb_gated_norm_update: null tensor");
+  QS_REQUIRE(groups >= 1 && width % groups == 0, "hyb_gated_norm_update: the width must split into `groups` equal parts");
+  QS_REQUIRE(dtype == QS_DTYPE_BF16 || dtype == QS_DTYPE_F32, "dtype must be QS_DTYPE_BF16 or QS_DTYPE_F32");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const int part = width / groups, chunks = (part + 3) / 4;
+  // warps per group: two chunks of four columns per lane where the block stays within 16 warps, up to eight otherwise
+  const int per = std::max(1, std::min((chunks + 63) / 64, 16 / groups));
+  const int nv = (chunks + per * 32 - 1) / (per * 32);
+  if (part % 4 == 0 && groups <= 16 && nv <= 8 && al16(out_h) && al16(x) && al16(add) && al16(add_bias) && al16(gate_bias) && al16(w) && al16(w_next) &&
+      al16(gate) && gate_stride % 4 == 0) {
+    const int threads = groups * per * 32;
+#define QS_GNU(ST, NV)                                                                                                                            \
+  gated_norm_update_vec_kernel<ST, NV><<<tokens_n, threads, 0, s>>>((ST*)out_h, x, fresh, add, add_f32, add_bias, (const ST*)gate, gate_stride,    \
+                                                                    gate_bias, w, mult, w_next, groups, offset, eps, width)
+#define QS_GNU_NV(ST)                        \
+  do {                                       \
+    if (nv <= 1) QS_GNU(ST, 1);              \
+    else if (nv <= 2) QS_GNU(ST, 2);         \
+    else if (nv <= 4) QS_GNU(ST, 4);         \
+    else QS_GNU(ST, 8);                      \
+  } while (0)
+    QS_DT(dtype, QS_GNU_NV(__nv_bfloat16), QS_GNU_NV(float));
+#undef QS_GNU_NV
+#undef QS_GNU
+    return check_cuda(cudaGetLastError(), "hyb_gated_norm_update");
+  }
+  const size_t smb = ((size_t)width + groups) * sizeof(float);
+  QS_REQUIRE(smb <= 200 * 1024, "hyb_gated_norm_update: row too wide for shared memory");
+#define QS_GNU(ST)                                                                                                                            \
+  do {                                                                                                                                        \
+    if (smb > 48 * 1024) cudaFuncSetAttribute(gated_norm_update_kernel<ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smb);           \
+    gated_norm_update_kernel<ST><<<tokens_n, 256, smb, s>>>((ST*)out_h, x, fresh, add, add_f32, add_bias, (const ST*)gate, gate_stride,      \
+                                                            gate_bias, w, mult, w_next, groups, offset, eps, width);                         \
+  } while (0)
+  QS_DT(dtype, QS_GNU(__nv_bfloat16), QS_GNU(float));
+#undef QS_GNU
+  return check_cuda(cudaGetLastError(), "hyb_gated_norm_update");
 }
 
 int qs_hyb_cast_rows(void* out, const float* x, int64_t n, int dtype, void* stream) {

@@ -120,8 +120,41 @@ struct AttnExtra {
   const float* slopes;
   const void* gate;
   long long gate_stride;
+  int gate_wide;
+  float softcap;
 };
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// the same on the special-function unit (relative error about 2^-21): for gates read from bfloat16 rows
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + fast_exp2(-1.4426950408889634f * fmaxf(z, -80.f))); }
+
+// Scores of a warp's tile, capped: s <- out * tanh(in * s), fp32.  While every |in * s| of the warp is at most 1/4 (scores well below the cap)
+// the tanh is its power series through u^9 (the first term left out is below 1e-8 of u there); otherwise tanh u = 1 - 2 / (1 + e^(2u)) on the
+// special-function unit, absolute error near 2^-22.  Every lane of the warp takes part.
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&s)[N][4], float in, float out) {
+  float top = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      s[i][j] *= in;
+      top = fmaxf(top, fabsf(s[i][j]));
+    }
+  if (__any_sync(0xffffffffu, top > 0.25f)) {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] = out - __fdividef(2.f * out, 1.f + fast_exp2(2.f * 1.4426950408889634f * fminf(s[i][j], 40.f)));
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float u = s[i][j], q = u * u;
+        s[i][j] = out * u * (1.f + q * (-1.f / 3.f + q * (2.f / 15.f + q * (-17.f / 315.f + q * (62.f / 2835.f)))));
+      }
+  }
+}
 
 }  // namespace hyb
 }  // namespace qs

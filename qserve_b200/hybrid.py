@@ -4,8 +4,9 @@ paged cache, or a recurrent layer over a state slot) beside an optional feed-for
 The model is assembled from a `HybridConfig` (qserve_b200.modelcfg): mixers are looked up in `MIXERS` and feed-forwards in `FEED_FORWARDS`
 by config type, so another design reuses them with other constants.  Layers are "parallel" blocks (mixer and feed-forward read the same
 stream and their output projections are one product), "sequential" blocks (mixer, then feed-forward) on one or several residual streams
-with learned read / write / mixing coefficients, or "post" blocks (mixer, then feed-forward, each taking the un-normed stream and normed on the
-way back, with a learned scale per channel).  A forward pass takes a `StepBatch` -- the flat batch a scheduler step has put together (portions of
+with learned read / write / mixing coefficients, "post" blocks (mixer, then feed-forward, each taking the un-normed stream and normed on the
+way back, with a learned scale per channel), or "sandwich" blocks (mixer, then feed-forward, each normed on the way in and on the way back, with
+a gate on what it puts out).  A forward pass takes a `StepBatch` -- the flat batch a scheduler step has put together (portions of
 prompts beside single decoded tokens) -- and the `HybridCache`; there is no other forward path: whole prompts, portions and decoding
 all go through `HybridDecoder.forward`.
 
@@ -15,7 +16,7 @@ Matrix products are cuBLAS through torch (as the quantised models' lm_head is); 
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Sequence
 
 import torch
@@ -92,12 +93,10 @@ class StepBatch:
     long_tokens: Optional[torch.Tensor] = None   # int32 [n_long] rows covered by tiles
     short_tokens: Optional[torch.Tensor] = None  # int32 [n_short] all other rows
 
-    # entries of at least TILE_MIN tokens, when `build` is told the page size: their sequences' pages so far, numbered in one run, so that a
-    # mixer can lay out per-step copies of what those pages hold (page i of the run is the sequence's page ctx_src[i]; ctx_table is a block
-    # table into the run)
-    n_ctx_pages: int = 0
-    ctx_src: Optional[torch.Tensor] = None     # int64 [n_ctx_pages] page of the pool
-    ctx_table: Optional[torch.Tensor] = None   # int32 [slots, max_blocks]
+    # when `build` is told the page size: (slot, first position, tokens) of the entries of at least TILE_MIN tokens, for `context`
+    page_size: int = 0
+    long_spans: Sequence[tuple] = ()
+    _contexts: dict = field(default_factory=dict)
 
     TILE_MIN = 16
     TILE_ROWS = 64
@@ -148,19 +147,29 @@ class StepBatch:
             host = host.pin_memory()
         b = StepBatch.view(host.to(device, non_blocking=True), sizes, block_table)
         if page_size > 0:
-            slots, idx = [], []
-            for s, p0, _, toks in entries:
-                if len(toks) >= StepBatch.TILE_MIN:
-                    n = -(-(p0 + len(toks)) // page_size)
-                    slots += [s] * n
-                    idx += range(n)
-            if slots:
-                cs, ci = torch.tensor(slots, dtype=torch.int64).to(device), torch.tensor(idx, dtype=torch.int64).to(device)
-                b.n_ctx_pages = len(slots)
-                b.ctx_src = block_table[cs, ci].to(torch.int64)
-                b.ctx_table = torch.zeros_like(block_table)
-                b.ctx_table[cs, ci] = torch.arange(len(slots), dtype=block_table.dtype, device=device)
+            b.page_size = page_size
+            b.long_spans = [(s, p0, len(toks)) for s, p0, _, toks in entries if len(toks) >= StepBatch.TILE_MIN]
         return b
+
+    def context(self, chunk: int = 0, window: int = 0):
+        """The pages that the entries of at least TILE_MIN tokens may look at under a mask, numbered in one run, so that a mixer can lay out
+        per-step copies of what they hold: (page of the pool of every page of the run int64 [n], block table into the run), or None without
+        such entries.  A page before an entry's first visible position (rounded down to a key tile of TILE_ROWS) is not part of the run."""
+        if not self.long_spans:
+            return None
+        if (chunk, window) not in self._contexts:
+            slots, idx = [], []
+            for s, p0, n in self.long_spans:
+                first = max(p0 - p0 % chunk if chunk > 0 else 0, p0 - window + 1 if window > 0 else 0)
+                span = range(first // self.TILE_ROWS * self.TILE_ROWS // self.page_size, -(-(p0 + n) // self.page_size))
+                slots += [s] * len(span)
+                idx += span
+            dev = self.block_table.device
+            cs, ci = torch.tensor([slots, idx], dtype=torch.int64).to(dev)
+            table = torch.zeros_like(self.block_table)
+            table[cs, ci] = torch.arange(len(slots), dtype=table.dtype, device=dev)
+            self._contexts[(chunk, window)] = (self.block_table[cs, ci].to(torch.int64), table)
+        return self._contexts[(chunk, window)]
 
 
 # ------------------------------------------------------------------------------------------------------------------------
@@ -174,9 +183,11 @@ class _Mixer:
         """Keep the output projection on the device (blocks that do not fold it into a product of their own)."""
         self.w_out = st(self.w_out)
 
-    def project(self, cat: torch.Tensor, dt: int, stream):
-        """Head outputs -> the mixer's output rows [T, W]; returns (rows, rows are fp32)."""
-        return torch.mm(cat, self.w_out.t()), False
+    out_bias: Optional[torch.Tensor] = None  # fp32 [W]; added by the block where it takes the rows
+
+    def project(self, cat: torch.Tensor, dt: int, stream, f32: bool = False):
+        """Head outputs -> the mixer's output rows [T, W] (f32: the product's accumulator as it is); returns (rows, rows are fp32)."""
+        return (_mm_f32(cat, self.w_out.t()), True) if f32 else (torch.mm(cat, self.w_out.t()), False)
 
 
 class MultiMapAttentionMixer(_Mixer):
@@ -184,18 +195,23 @@ class MultiMapAttentionMixer(_Mixer):
     o = a1 - lambda a2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, then unit RMS per head and a factor (1 - diff).
     With one map: optional projection biases, unit-RMS q / k (with gains shared by the heads), a learned temperature per head (folded into the
     prepared query), a sink term in the denominator, a mask by chunks of positions and / or a window that may keep the sequence's first
-    positions visible, a linear distance bias per head, values tied to the key projection's raw output (no value projection), and a sigmoid gate per head
-    (its logits are the last `heads` columns of the mixer's projection rows)."""
+    positions visible, a tanh cap on the scores, a linear distance bias per head, values tied to the key projection's raw output (no value
+    projection) or brought to unit RMS per head before they are cached, an output bias, and a sigmoid gate per head or per output number (its
+    logits are the last columns of the mixer's projection rows)."""
 
     def __init__(self, m: AttentionMixerConfig, w: Dict[str, torch.Tensor], eps: float, dtype, device):
         self.m, self.eps = m, eps
         assert m.heads % m.kv_heads == 0
         f32 = lambda t: t.to(torch.float32).to(device).contiguous()
-        self.general = m.rot is None or m.rot.layout != "interleaved" or m.bias or m.qk_norm or m.head_temp or m.tied_values
-        plus = m.sink or m.keep_first or m.distance_slope > 0.0 or m.head_gate or m.qk_gain
+        self.general = m.rot is None or m.rot.layout != "interleaved" or m.bias or m.qk_norm or m.head_temp or m.tied_values or m.value_norm
+        plus = m.sink or m.keep_first or m.distance_slope > 0.0 or m.head_gate or m.qk_gain or m.gate_wide or m.softcap > 0.0 or m.sink_score is not None
         if (self.general or plus) and m.maps != 1:
-            raise ValueError("biases, unit-RMS q / k, head temperatures, sinks, kept first positions, distance biases, tied values, head gates and "
-                             "non-interleaved rotations need one score map per head")
+            raise ValueError("biases, unit-RMS q / k / v, head temperatures, sinks, kept first positions, score caps, distance biases, tied values, "
+                             "gates and non-interleaved rotations need one score map per head")
+        if m.sink and m.sink_score is not None or m.head_gate and m.gate_wide:
+            raise ValueError("a learned sink or a fixed one, a gate per head or one per output number")
+        if m.softcap < 0.0 or m.softcap > 0.0 and m.scale <= 0.0:
+            raise ValueError("a score cap is positive and goes with a positive scale")
         if m.keep_first and (m.window <= 0 or m.chunk):
             raise ValueError("kept first positions go with a window and no chunks")
         if m.tied_values and m.vdim != m.dim:
@@ -211,14 +227,19 @@ class MultiMapAttentionMixer(_Mixer):
         self.slopes = torch.tensor(sl, dtype=torch.float64).to(torch.float32).to(device) if sl is not None else None
         self.temp = f32(w["temp"]) if m.head_temp else None
         self.sinks = f32(w["sink"]) if m.sink else None
+        if m.sink_score is not None:
+            self.sinks = torch.full((m.heads,), float(m.sink_score), dtype=torch.float32, device=device)
+        self.out_bias = f32(w["o.b"]) if m.out_bias else None
         for t, n in ((self.temp, "temp"), (self.sinks, "sink")):
             if t is not None and t.numel() != m.heads:
                 raise ValueError(f"attention weight {n} must have one number per head")
         self.col_g = (m.heads + m.kv_heads) * m.maps * m.dim + (0 if m.tied_values else m.kv_heads * m.vdim)
-        self.in_features = self.col_g + (m.heads if m.head_gate else 0)
         self.out_features = m.heads * m.vdim
-        rows_of = {"q": m.heads * m.maps * m.dim, "k": m.kv_heads * m.maps * m.dim, "v": m.kv_heads * m.vdim, "g": m.heads}
-        parts += ["g"] if m.head_gate else []
+        rows_of = {"q": m.heads * m.maps * m.dim, "k": m.kv_heads * m.maps * m.dim, "v": m.kv_heads * m.vdim, "g": self.out_features if m.gate_wide else m.heads}
+        gated = m.head_gate or m.gate_wide
+        parts += ["g"] if gated else []
+        self.extra = m.keep_first or self.slopes is not None or gated or m.softcap > 0.0  # something for the kernels' optional parts
+        self.gated = gated
         for name in parts:
             if w[name].shape[0] != rows_of[name]:
                 raise ValueError(f"attention weight {name}: {tuple(w[name].shape)} does not have {rows_of[name]} rows")
@@ -247,16 +268,16 @@ class MultiMapAttentionMixer(_Mixer):
         fast = scratch is not None and ATTENTION_IMPL != "plain" and \
             lib.qs_hyb_attention_fast_supported(dt, m.heads, m.kv_heads, m.maps, m.dim, m.vdim, proj.stride(0)) == 1
         extra = None
-        if m.keep_first or self.slopes is not None or m.head_gate:
-            gate = proj.data_ptr() + self.col_g * proj.element_size() if m.head_gate else None
-            extra = ctypes.byref(AttnExtra(m.keep_first, _p(self.slopes), gate, proj.stride(0)))
+        if self.extra:
+            gate = proj.data_ptr() + self.col_g * proj.element_size() if self.gated else None
+            extra = ctypes.byref(AttnExtra(m.keep_first, _p(self.slopes), gate, proj.stride(0), 1 if m.gate_wide else 0, m.softcap))
         if self.general:
             check(lib.qs_hyb_qk_prepare_append(proj.data_ptr(), proj.stride(0), _p(self.bias), _p(self.temp), _p(b.tok_slot), _p(b.tok_pos),
                                                _p(b.block_table), b.block_table.shape[1], run_cache["k"].data_ptr(), run_cache["v"].data_ptr(),
                                                _p(self.inv_freq), 1 if m.rot is not None and m.rot.layout == "half" else 0,
                                                m.rot.dims if m.rot is not None else 0, 1 if m.qk_norm else 0, self.eps, b.n_tokens, m.heads,
                                                m.kv_heads, m.dim, m.vdim, page_size, _p(self.q_gain), _p(self.k_gain), 1 if m.tied_values else 0,
-                                               dt, stream))
+                                               1 if m.value_norm else 0, dt, stream))
         else:
             check(lib.qs_hyb_rope_append(proj.data_ptr(), proj.stride(0), _p(b.tok_slot), _p(b.tok_pos), _p(b.block_table), b.block_table.shape[1],
                                          run_cache["k"].data_ptr(), run_cache["v"].data_ptr(), self.inv_freq.data_ptr(), self.amp, b.n_tokens,
@@ -482,7 +503,8 @@ class LatentAttentionMixer(_Mixer):
         fast = scratch is not None and LATENT_IMPL != "plain" and lib.qs_hyb_latent_attention_fast_supported(dt, H, K, R) == 1
         # portions of at least StepBatch.TILE_MIN tokens: per-head keys and values (less arithmetic per score than the K + R numbers of a cell);
         # single tokens and short portions: queries taken to the latent, scored against the cells as they lie
-        per_head = scratch is not None and self.per_head_ok and LATENT_IMPL not in ("plain", "latent") and b.n_tiles > 0 and b.n_ctx_pages > 0
+        ctx = b.context(m.chunk, m.window) if scratch is not None and self.per_head_ok and LATENT_IMPL not in ("plain", "latent") and b.n_tiles > 0 else None
+        per_head = ctx is not None
         latent = not per_head or b.n_short > 0
         qa = olat = ov = otok = None
         if latent:
@@ -491,14 +513,19 @@ class LatentAttentionMixer(_Mixer):
         check(lib.qs_hyb_latent_query(_p(qa), qlat.data_ptr() if latent else None, q.data_ptr(), q.stride(0), _p(self.inv_freq), self.rot_dims,
                                       _p(b.tok_pos), T, H, D, K, R, 1 if per_head else 0, self.rot_layout, self.amp, dt, stream))
         if per_head:
-            cells = pool.index_select(0, b.ctx_src).view(-1, K + R)
+            ctx_src, ctx_table = ctx
+            cells = pool.index_select(0, ctx_src).view(-1, K + R)
             keys, values = torch.mm(cells, self.w_keys.t()), torch.mm(cells[:, :K], self.w_values.t())
-            otok = torch.empty((T, H * Dv), dtype=proj.dtype, device=dev)
+            # without single tokens and gates the heads' outputs are already what the output projection reads
+            direct = not latent and not m.gate
+            otok = out if direct else torch.empty((T, H * Dv), dtype=proj.dtype, device=dev)
             check(lib.qs_hyb_attention_fast(otok.data_ptr(), otok.stride(0), q.data_ptr(), q.stride(0), keys.data_ptr(), values.data_ptr(), _p(b.tok_slot),
-                                            _p(b.tok_pos), b.ctx_table.data_ptr(), b.ctx_table.shape[1], _p(b.tile_entry), _p(b.tile_row0), b.n_tiles,
+                                            _p(b.tok_pos), ctx_table.data_ptr(), ctx_table.shape[1], _p(b.tile_entry), _p(b.tile_row0), b.n_tiles,
                                             _p(b.long_tokens), b.n_long, None, 0, _p(b.entry_start), _p(b.entry_len), _p(b.entry_slot), _p(b.entry_pos0),
                                             scratch.data_ptr(), H, H, 1, D + R, Dv, m.scale, 0.0, 1.0, self.eps, 0, page_size, m.chunk, m.window,
                                             _p(self.sinks), None, dt, stream))
+            if direct:
+                return
         if latent:
             olat = torch.empty((H, T, K), dtype=proj.dtype, device=dev)
             if fast:
@@ -547,12 +574,12 @@ class ParallelMixer(_Mixer):
         self.left.run(proj[:, :a], out[:, :oa], b, run_cache["left"], page_size, scratch, dt, stream)
         self.right.run(proj[:, a:], out[:, oa:], b, run_cache["right"], page_size, scratch, dt, stream)
 
-    def project(self, cat: torch.Tensor, dt: int, stream):
+    def project(self, cat: torch.Tensor, dt: int, stream, f32: bool = False):
         oa = self.left.out_features
         yl, fl = self.left.project(cat[:, :oa], dt, stream)
         yr, fr = self.right.project(cat[:, oa:], dt, stream)
-        if fl or fr:
-            raise NotImplementedError("side-by-side mixers whose own outputs are fp32 rows")
+        if fl or fr or self.left.out_bias is not None or self.right.out_bias is not None:
+            raise NotImplementedError("side-by-side mixers whose own outputs are fp32 rows or have biases")
         T, W = yl.shape
         y = torch.empty((T, W), dtype=torch.float32, device=cat.device)
         check(lib.qs_hyb_branch_norm_mean(y.data_ptr(), yl.data_ptr(), yr.data_ptr(), self.gain_left.data_ptr(), self.gain_right.data_ptr(),
@@ -676,12 +703,15 @@ class DenseFeedForward:
                 raise ValueError("dense feed-forward: the biases do not match their projections")
 
     def run(self, h: torch.Tensor, dt: int, stream):
-        gu = torch.mm(h, self.w_in.t())
-        act = torch.empty((h.shape[0], self.ff), dtype=h.dtype, device=h.device)
-        if self.in_bias is None and self.act == 0:
-            check(lib.qs_hyb_gelu_tanh_mul(act.data_ptr(), act.stride(0), gu.data_ptr(), h.shape[0], self.ff, dt, stream))
+        return self.finish(torch.mm(h, self.w_in.t()), dt, stream)
+
+    def finish(self, gu: torch.Tensor, dt: int, stream):
+        """From the rows [gate | up (| columns of somebody else)] of the input product on."""
+        act = torch.empty((gu.shape[0], self.ff), dtype=gu.dtype, device=gu.device)
+        if self.in_bias is None and self.act == 0 and gu.stride(0) == 2 * self.ff:
+            check(lib.qs_hyb_gelu_tanh_mul(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.shape[0], self.ff, dt, stream))
         else:
-            check(lib.qs_hyb_bias_gated_act(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), _p(self.in_bias), h.shape[0], self.ff, self.act, dt,
+            check(lib.qs_hyb_bias_gated_act(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), _p(self.in_bias), gu.shape[0], self.ff, self.act, dt,
                                             stream))
         return _mm_f32(act, self.w_down.t()), True
 
@@ -709,11 +739,15 @@ class _Layer:
         self.norm1_b = self.norm2_b = self.mlp_in_bias = self.out_bias = self.side_ff = None
         self.w_all_in = None  # mixer and feed-forward input projections stacked (blocks whose branches read one normed row)
         self.gated = True
+        # sandwich blocks: gains of the norms on the way back, biases of the residual gates, and the sublayers' stacked input projections (mixer /
+        # feed-forward rows first, then the gate's rows from column gate1 / gate2 on)
+        self.norm1_back = self.norm2_back = self.gate1_b = self.gate2_b = self.w_mix_in = self.w_ff_in = None
+        self.gate1 = self.gate2 = 0
         self.ls1 = self.ls2 = None  # post-norm blocks: per-channel scales of the normed sublayer outputs
 
 
 class HybridDecoder:
-    """Two block forms (HybridConfig.block):
+    """Block forms (HybridConfig.block):
 
     "parallel":   x <- x + (mixer(norm1 x) + ff(norm2 x)) per layer run, both branches of the same x; the two output projections are ONE
                   product: [mixer heads | ff activation] @ [W_o | W_down]^T, so the sum of the branches is accumulated in fp32 inside the GEMM.
@@ -722,7 +756,10 @@ class HybridDecoder:
                   the streams happens inside the next sublayer's norm kernel.
     "post":       x <- x + ls1 norm1(mixer(x)), then x <- x + ls2 norm2(ff(x)): a sublayer takes the un-normed stream (its storage-type copy is
                   written by the kernel that lands the previous sublayer), and its fp32 output rows are normed, scaled per channel and
-                  added in one kernel."""
+                  added in one kernel.
+    "sandwich":   x <- x + m norm1b(g1 * mixer(h)), h = norm1 x, then x <- x + m norm2b(g2 * ff(h)), h = norm2 x, with g = sigmoid(W h + b) per channel
+                  (`residual_gate`).  A gate's rows ride in its sublayer's input product; ONE kernel lands the sublayer (bias, gate, norm,
+                  residual in fp32) and norms the stream for the next one."""
 
     def __init__(self, cfg: HybridConfig, weights: Dict[str, torch.Tensor], dtype: torch.dtype = torch.bfloat16, device: Optional[torch.device] = None):
         if dtype not in _DT:
@@ -744,10 +781,18 @@ class HybridDecoder:
         if self.pair is not None and self.pair.shape[0] != cfg.pair_buckets + 1:
             raise ValueError("the pair table must have buckets + 1 rows")
         self.head = st(weights["head"])
+        # a factor on the logits rides in the last norm's gain
         self.final_norm = f32(weights["final.norm"])
+        if cfg.logit_scale != 1.0:
+            self.final_norm = (cfg.norm_offset + self.final_norm) * cfg.logit_scale - cfg.norm_offset
         self.layers: List[_Layer] = []
-        if cfg.block not in ("parallel", "sequential", "post"):
+        if cfg.block not in ("parallel", "sequential", "post", "sandwich"):
             raise ValueError(f"unknown block form {cfg.block!r}")
+        if cfg.block != "sandwich" and (cfg.residual_gate or cfg.embed_norm or cfg.residual_mult != 1.0):
+            raise NotImplementedError("residual gates, a residual factor and a normed embedding are built for sandwich blocks")
+        if cfg.norm_groups < 1 or W % cfg.norm_groups:
+            raise ValueError("norm groups must divide the width")
+        self.embed_norm = f32(weights["embed.norm"]) if cfg.embed_norm else None
         self.n_streams = max(cfg.streams, 1) if cfg.block == "sequential" else 1
         one = torch.ones(1, dtype=torch.float32, device=dev)
 
@@ -763,6 +808,11 @@ class HybridDecoder:
             pre = f"l{i}."
             mw = {k[len(pre) + 4:]: v for k, v in weights.items() if k.startswith(pre + "mix.")}
             mixer = MIXERS[type(ly.mixer)](ly.mixer, mw, cfg.eps, dtype, dev)
+            if mixer.out_bias is not None and (cfg.block not in ("post", "sandwich") or mixer.out_bias.numel() != W):
+                raise ValueError("an output bias has `width` numbers and goes with post-norm and sandwich blocks")
+            if cfg.block == "sandwich":
+                self.layers.append(self._sandwich_layer(ly, mixer, weights, pre, st, f32))
+                continue
             if cfg.block == "post":
                 mixer.place_out(st)
                 ff = norm2 = None
@@ -830,7 +880,7 @@ class HybridDecoder:
             raise ValueError(f"unknown norm {cfg.norm_kind!r}")
         if cfg.norm_kind == "layer" and (cfg.block != "parallel" or cfg.norm_offset != 0.0 or cfg.norm_groups != 1):
             raise NotImplementedError("layer norms are built for parallel blocks with plain gains")
-        self.final_norm_b = f32(weights["final.norm.b"]) if cfg.norm_kind == "layer" else None
+        self.final_norm_b = f32(weights["final.norm.b"]) * cfg.logit_scale if cfg.norm_kind == "layer" else None
         self.loop_in = None
         if cfg.loop_in and cfg.pass_starts():
             self.loop_in = st(weights["loop.in"])
@@ -838,6 +888,38 @@ class HybridDecoder:
                 raise ValueError("loop.in must be [width, 2 width]")
         self.schedule = cfg.schedule()
         self._scratch: Optional[torch.Tensor] = None
+
+    def _sandwich_layer(self, ly, mixer, weights, pre: str, st, f32) -> _Layer:
+        cfg, W = self.cfg, self.cfg.width
+        mixer.place_out(st)
+        layer = _Layer(mixer, f32(weights[pre + "norm1"]), None, None, None, None)
+        layer.norm1_back = f32(weights[pre + "norm1b"])
+
+        def stacked(rows, gate):  # (input projection, column of the gate's rows, the gate's bias)
+            if not cfg.residual_gate:
+                return rows, 0, None
+            w, b = weights[pre + gate], f32(weights[pre + gate + ".b"])
+            if tuple(w.shape) != (W, W) or b.numel() != W:
+                raise ValueError(f"{pre}{gate}: a residual gate is [width, width] with a bias of width numbers")
+            rows = _pad_rows(rows)
+            return _pad_rows(torch.cat([rows, st(w)], 0)).contiguous(), rows.shape[0], b
+
+        layer.w_mix_in, layer.gate1, layer.gate1_b = stacked(mixer.w_in, "rg1")
+        del mixer.w_in
+        if ly.mlp is not None:
+            fw = {k[len(pre) + 4:]: v for k, v in weights.items() if k.startswith(pre + "mlp.")}
+            layer.ff = FEED_FORWARDS[type(ly.mlp)](ly.mlp, fw, W, self.dtype, self.device)
+            layer.norm2, layer.norm2_back = f32(weights[pre + "norm2"]), f32(weights[pre + "norm2b"])
+            if isinstance(layer.ff, DenseFeedForward):
+                layer.w_ff_in, layer.gate2, layer.gate2_b = stacked(layer.ff.w_in, "rg2")
+                del layer.ff.w_in
+            else:  # a feed-forward with input products of its own: the gate is a product beside it
+                none = torch.empty((0, W), dtype=self.dtype, device=self.device)
+                layer.w_ff_in, layer.gate2, layer.gate2_b = stacked(none, "rg2")
+        for t in (layer.norm1, layer.norm2, layer.norm1_back, layer.norm2_back):
+            if t is not None and t.numel() != W:
+                raise ValueError(f"{pre}: norm gains have `width` numbers")
+        return layer
 
     @classmethod
     def from_dir(cls, model_dir: str, dtype: torch.dtype = torch.bfloat16, device: Optional[torch.device] = None) -> "HybridDecoder":
@@ -872,6 +954,8 @@ class HybridDecoder:
             return self._forward_sequential(x, b, cache, tap, scratch, s)
         if cfg.block == "post":
             return self._forward_post(x, b, cache, tap, scratch, s)
+        if cfg.block == "sandwich":
+            return self._forward_sandwich(x, b, cache, tap, scratch, s)
         return self._forward_parallel(x, b, cache, tap, scratch, s)
 
     def _land(self, x, pending, s, out_h=None, w=None, bias=None, cat_out=None, x0=None) -> None:
@@ -980,11 +1064,47 @@ class HybridDecoder:
             cat = torch.empty((T, ly.mixer.out_features), dtype=self.dtype, device=dev)
             ly.mixer.run(proj, cat, b, cache.runs[run], cache.page_size, scratch, dt, s)
             y = _mm_f32(cat, ly.mixer.w_out.t())
-            check(lib.qs_hyb_post_norm_update(h_ptr, x.data_ptr(), y.data_ptr(), 1, None, ly.norm1.data_ptr(), _p(ly.ls1), cfg.norm_offset, cfg.eps, T, W, dt, s))
+            check(lib.qs_hyb_post_norm_update(h_ptr, x.data_ptr(), y.data_ptr(), 1, _p(ly.mixer.out_bias), ly.norm1.data_ptr(), _p(ly.ls1), cfg.norm_offset, cfg.eps, T, W, dt, s))
             if ly.ff is not None:
                 y, y32 = ly.ff.run(h, dt, s)
                 check(lib.qs_hyb_post_norm_update(h_ptr, x.data_ptr(), y.data_ptr(), 1 if y32 else 0, _p(getattr(ly.ff, "out_bias", None)),
                                                   ly.norm2.data_ptr(), _p(ly.ls2), cfg.norm_offset, cfg.eps, T, W, dt, s))
+            if tap is not None:
+                tap(run, x)
+        return x
+
+    def _sandwich_land(self, out_h, x, rows, rows_f32, bias, gate, gate_b, w, mult, w_next, s, fresh: bool = False) -> None:
+        """x <- [x +] mult norm(sigmoid(gate + gate_b) * (rows + bias)) w; the norm of x times w_next into out_h (None: not wanted)."""
+        cfg = self.cfg
+        check(lib.qs_hyb_gated_norm_update(_p(out_h), x.data_ptr(), 1 if fresh else 0, rows.data_ptr(), 1 if rows_f32 else 0, _p(bias), _p(gate),
+                                           gate.stride(0) if gate is not None else 0, _p(gate_b), w.data_ptr(), mult, _p(w_next), cfg.norm_groups,
+                                           cfg.norm_offset, cfg.eps, x.shape[0], cfg.width, self.dt, s))
+
+    def _forward_sandwich(self, x, b: StepBatch, cache: HybridCache, tap, scratch, s) -> torch.Tensor:
+        cfg, dev, dt, T, W = self.cfg, self.device, self.dt, b.n_tokens, self.cfg.width
+        h = torch.empty((T, W), dtype=self.dtype, device=dev)
+        layers = [self.layers[li] for li in self.schedule]
+        first = layers[0].norm1 if layers else None
+        if cfg.embed_norm:  # the stream starts as the normed embedding; its norm is the first sublayer's input
+            e, x = x, torch.empty_like(x)
+            self._sandwich_land(h if layers else None, x, e, True, None, None, None, self.embed_norm, 1.0, first, s, fresh=True)
+        elif layers:
+            check(lib.qs_hyb_stream_norm(h.data_ptr(), None, x.data_ptr(), 1, None, 0, None, None, None, first.data_ptr(), cfg.norm_groups, cfg.norm_offset,
+                                         cfg.eps, T, W, dt, s))
+        for run, ly in enumerate(layers):
+            after = layers[run + 1].norm1 if run + 1 < len(layers) else None  # gain of the norm the next layer reads; none after the last
+            rows = torch.mm(h, ly.w_mix_in.t())
+            cat = torch.empty((T, ly.mixer.out_features), dtype=self.dtype, device=dev)
+            ly.mixer.run(rows, cat, b, cache.runs[run], cache.page_size, scratch, dt, s)
+            y, y32 = ly.mixer.project(cat, dt, s, f32=True)
+            nxt = ly.norm2 if ly.ff is not None else after
+            self._sandwich_land(h if nxt is not None else None, x, y, y32, ly.mixer.out_bias, rows[:, ly.gate1:] if cfg.residual_gate else None, ly.gate1_b,
+                                ly.norm1_back, cfg.residual_mult, nxt, s)
+            if ly.ff is not None:
+                rows = torch.mm(h, ly.w_ff_in.t()) if ly.w_ff_in.shape[0] else None
+                y, y32 = ly.ff.finish(rows, dt, s) if isinstance(ly.ff, DenseFeedForward) else ly.ff.run(h, dt, s)
+                self._sandwich_land(h if after is not None else None, x, y, y32, getattr(ly.ff, "out_bias", None),
+                                    rows[:, ly.gate2:] if cfg.residual_gate else None, ly.gate2_b, ly.norm2_back, cfg.residual_mult, after, s)
             if tap is not None:
                 tap(run, x)
         return x
@@ -994,17 +1114,16 @@ class HybridDecoder:
         n, W = x_rows.shape
         x_rows = x_rows.contiguous()
         h = torch.empty((n, W), dtype=self.dtype, device=self.device)
-        if self.cfg.block == "sequential":
-            check(lib.qs_hyb_stream_norm(h.data_ptr(), None, x_rows.data_ptr(), 1, None, 0, None, None, None, self.final_norm.data_ptr(),
-                                         self.cfg.norm_groups, self.cfg.norm_offset, self.cfg.eps, n, W, self.dt, _stream(self.device)))
-            return torch.mm(h, self.head.t()).float()
         s = _stream(self.device)
-        if self.cfg.norm_kind == "rms":
+        if self.cfg.block in ("sequential", "sandwich"):
+            check(lib.qs_hyb_stream_norm(h.data_ptr(), None, x_rows.data_ptr(), 1, None, 0, None, None, None, self.final_norm.data_ptr(),
+                                         self.cfg.norm_groups, self.cfg.norm_offset, self.cfg.eps, n, W, self.dt, s))
+        elif self.cfg.norm_kind == "rms":
             check(lib.qs_hyb_rms_norm(h.data_ptr(), None, x_rows.data_ptr(), None, self.final_norm.data_ptr(), None, self.cfg.norm_offset, self.cfg.eps, n,
                                       W, self.dt, s))
         else:
             self._land(x_rows, None, s, out_h=h, w=self.final_norm, bias=self.final_norm_b)
-        out = _mm_f32(h, self.head.t()) if self.cfg.logit_softcap > 0.0 or self.cfg.block == "post" else torch.mm(h, self.head.t()).float()
+        out = _mm_f32(h, self.head.t()) if self.cfg.logit_softcap > 0.0 or self.cfg.block in ("post", "sandwich") else torch.mm(h, self.head.t()).float()
         if self.cfg.logit_softcap > 0.0:
             check(lib.qs_hyb_softcap(out.data_ptr(), out.numel(), self.cfg.logit_softcap, s))
         return out
@@ -1050,8 +1169,10 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
                 w[p + "v"] = r(G * Dv, W, s=W ** -0.5)
             if m.qk_gain:
                 w[p + "q.norm"], w[p + "k.norm"] = 1.0 + r(D, s=0.1), 1.0 + r(D, s=0.1)
-            if m.head_gate:
-                w[p + "g"] = r(H, W, s=W ** -0.5)
+            if m.head_gate or m.gate_wide:
+                w[p + "g"] = r(H * Dv if m.gate_wide else H, W, s=W ** -0.5)
+            if m.out_bias:
+                w[p + "o.b"] = r(W, s=0.1)
             if m.maps == 2:
                 for n in ("lq1", "lk1", "lq2", "lk2"):
                     w[p + n] = r(D, s=0.1)
@@ -1084,6 +1205,8 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
     gain = (lambda: 1.0 + r(W, s=0.1)) if cfg.norm_offset == 0.0 else (lambda: r(W, s=0.1))
     w = {"embed": r(cfg.vocab, W), "head": r(cfg.vocab, W, s=W ** -0.5), "final.norm": gain()}
     layer_norm = cfg.norm_kind == "layer"
+    if cfg.embed_norm:
+        w["embed.norm"] = gain()
     if layer_norm:
         w["final.norm.b"] = r(W, s=0.1)
     if cfg.loop_in:
@@ -1117,6 +1240,11 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
                     w[p + "mlp.up.b"], w[p + "mlp.down.b"] = r(ly.mlp.ff, s=0.1), r(W, s=0.1)
                     if ly.mlp.gated:
                         w[p + "mlp.gate.b"] = r(ly.mlp.ff, s=0.1)
+        if cfg.block == "sandwich":
+            for q in (1, 2) if ly.mlp is not None else (1,):
+                w[f"{p}norm{q}b"] = gain()
+                if cfg.residual_gate:
+                    w[f"{p}rg{q}"], w[f"{p}rg{q}.b"] = r(W, W, s=W ** -0.5), r(W, s=0.1)
         if cfg.layer_scale:
             w[p + "ls1"] = 0.5 + r(W, s=0.05)
             if ly.mlp is not None:

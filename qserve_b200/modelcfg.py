@@ -97,6 +97,11 @@ class AttentionMixerConfig:
     tied_values: bool = False  # no value projection: a position's value is the key projection's output (bias included), taken ahead of the unit-RMS step
     distance_slope: float = 0.0  # > 0: slope_h (i - j) is taken off the score of query i and key j, slope_h = 2^(-distance_slope (h + 1) / heads)
     head_gate: bool = False  # head h's output is multiplied by sigmoid((W_g x)_h) (tensor g [heads, width])
+    gate_wide: bool = False  # the heads' outputs are multiplied entry by entry by sigmoid(W_g x) (tensor g [heads * vdim, width])
+    softcap: float = 0.0     # > 0: a scaled score s becomes softcap * tanh(s / softcap), ahead of the distance bias
+    value_norm: bool = False  # value heads are brought to unit RMS before they are cached
+    sink_score: Optional[float] = None  # the softmax denominator has one more term exp(sink_score) without a value, the same for every head
+    out_bias: bool = False   # the output projection has a bias (tensor o.b)
 
     def slopes(self):
         """Per-head slope of the distance bias (float64 list), or None."""
@@ -239,6 +244,7 @@ class HybridConfig:
     norm_offset: float = 1.0  # gains are stored as offsets from this value
     block: str = "parallel"   # "parallel": x += mixer(norm1 x) + ff(norm2 x);  "sequential": x += mixer(norm1 x), then x += ff(norm2 x);
                               # "post": x += ls1 norm1(mixer(x)), then x += ls2 norm2(ff(x)): the un-normed stream goes into a sublayer, what comes out is normed
+                              # "sandwich": x += m norm1b(g1 mixer(norm1 x)), then x += m norm2b(g2 ff(norm2 x)), m = residual_mult, g1 / g2 optional gates
     streams: int = 0          # sequential blocks: > 0 = that many residual streams with hyper-connection coefficients (tensors hc1.*, hc2.*)
     norm_groups: int = 1      # RMS norms work on this many equal consecutive parts of the width, each with its own statistic
     embed_scale: float = 1.0
@@ -246,6 +252,10 @@ class HybridConfig:
     shared_norm: bool = False  # parallel blocks: the mixer and the feed-forward read ONE normed row (norm1; there is no norm2)
     loop_in: bool = False     # before the first layer of every pass of the loop: x <- W [x; x0] (tensor loop.in [W, 2 W], x0 the embedding output)
     logit_softcap: float = 0.0  # > 0: logits <- cap * tanh(logits / cap)
+    residual_mult: float = 1.0  # "sandwich" blocks: factor of a normed sublayer output
+    residual_gate: bool = False  # "sandwich" blocks: a sublayer's output times sigmoid(W h + b) of its input h, ahead of its norm (tensors rg1, rg1.b, rg2, rg2.b)
+    embed_norm: bool = False    # "sandwich" blocks: the embedding is normed (tensor embed.norm)
+    logit_scale: float = 1.0    # logits <- logit_scale * head x, ahead of a cap
     layer_scale: bool = False   # "post" blocks: a normed sublayer output is multiplied per channel by a learned row (tensors ls1, ls2)
 
     def schedule(self):
@@ -404,9 +414,44 @@ def parse_zuzezen(c: dict) -> HybridConfig:
                         embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)), layer_scale=True)
 
 
+def parse_nagosun(c: dict) -> HybridConfig:
+    """Nagosun: sandwich blocks (a sublayer's input and its gated output are both RMS-normed in equal groups of channels; the sum is weighed by a
+    constant), a normed embedding, scaled logits; mixers `attention` (grouped heads with biases, unit-RMS values, capped scores less a
+    linear distance bias, a sliding window, a sink of fixed score 0, a sigmoid gate per output number) and `latent_attention`
+    (queries projected directly, interleaved rotary pairs on the shared rotated part, a sliding window); dense silu-gated feed-forwards."""
+    layers = []
+    for ly in c["layers"]:
+        m = ly["mixer"]
+        window = int((m.get("mask") or {}).get("size", 0))
+        if ly["type"] == "attention":
+            mixer = AttentionMixerConfig(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]), int(m.get("vdim", m["dim"])), None,
+                                         float(m["scale"]), bias=True, window=window, distance_slope=8.0, gate_wide=True,
+                                         softcap=float(m.get("softcap") or 0.0), value_norm=True, sink_score=0.0, out_bias=True)
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError("kv_heads must divide heads")
+        elif ly["type"] == "latent_attention":
+            rot = _parse_rot(m["rot"]) if m.get("rot") else None
+            mixer = LatentAttentionMixerConfig(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), 0, rot,
+                                               float(m["scale"]), gate=False, window=window)
+            if rot is not None and (rot.dims > mixer.rot_dim or rot.dims % 2):
+                raise ValueError("latent attention rotates an even number of at most rot_dim entries")
+        else:
+            raise ValueError(f"unknown mixer type {ly['type']!r}")
+        mlp = ly.get("mlp")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"unknown feed-forward kind {mlp.get('kind')!r}")
+        layers.append(HybridLayerConfig(ly["type"], mixer, MlpConfig("dense", int(mlp["ff"]), act="silu") if mlp is not None else None))
+    groups = int(c["norm"].get("groups", 1))
+    if groups < 1 or int(c["width"]) % groups:
+        raise ValueError("norm groups must divide the width")
+    return HybridConfig("Nagosun", int(c["vocab"]), int(c["width"]), float(c["norm"]["eps"]), tuple(layers), norm_offset=0.0, block="sandwich",
+                        norm_groups=groups, residual_mult=float(c.get("residual_mult", 1.0)), residual_gate=True, embed_norm=True,
+                        logit_scale=float(c.get("logit_scale", 1.0)))
+
+
 # config.json "architecture" -> parser.  The quantised Llama-family models of MODELS are built by qserve_b200.decode.DecodeRunner.
 ARCHITECTURES: Dict[str, Callable[[dict], HybridConfig]] = {"Rizurax": parse_rizurax, "Toderax": parse_toderax, "Nusuvik": parse_nusuvik,
-                                                                 "Zuzezen": parse_zuzezen}
+                                                                 "Zuzezen": parse_zuzezen, "Nagosun": parse_nagosun}
 
 
 def read_model_config(model_dir: str) -> HybridConfig:
