@@ -16,6 +16,7 @@ is Qwen1.5-72B (all 80 layers) tensor-parallel over the N GPU
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
 import math
 import os
@@ -69,6 +70,10 @@ def parse():
                     "(post-norm blocks, gated linear attention, windowed attention with tied values and a distance bias, latent attention with a "
                     "sink; random weights) at layer sizes of real models, beside the Rizurax hybrid decoder at equal size and its like kernels "
                     "in the other designs; prints one JSON line")
+    ap.add_argument("--nagosun", action="store_true", help="instead of the default workload: prefill and decode throughput of the Nagosun decoder "
+                    "(sandwich blocks with grouped norms and residual gates, windowed attention with capped scores and unit-RMS values, windowed "
+                    "latent attention; random weights) at layer sizes of real models, beside the Zuzezen decoder at equal size and its like "
+                    "kernels; prints one JSON line")
     return ap.parse_args()
 
 
@@ -1138,6 +1143,61 @@ def nusuvik_block(args):
 
 
 # ------------------------------------------------------------------------------------------------------------
+# parts that the hybrid decoders' options share: whole steps on an engine, one mixer on an engine's batches, a mixer of another design
+# ------------------------------------------------------------------------------------------------------------
+HYBRID_LOAD = (64, 1024, 4, 2048)  # decode batch and context, prompts and their length
+
+
+def hybrid_steps(model, eng, V, g, reps, stream):
+    """Prefill (all prompts in one step) and decode of HYBRID_LOAD -> (record, prompt batch, decode batch)."""
+    import torch
+
+    from qserve_b200.hybrid import StepBatch
+
+    (B, CTX, NP, LP), dev = HYBRID_LOAD, model.device
+    prompts = [torch.randint(0, V, (LP,), generator=g).tolist() for _ in range(NP)]
+    for i, p_ in enumerate(prompts):
+        eng.cache.admit(("p", i)); eng.cache.reserve(("p", i), LP)
+    pb = StepBatch.build([(eng.cache.seqs[("p", i)].slot, 0, -1, p_) for i, p_ in enumerate(prompts)], eng.cache.sync_block_table(), dev,
+                         eng.cache.page_size)
+    t = time_kernel(lambda: (model.forward(pb, eng.cache), 1)[1], reps, stream)
+    rec = {"prefill": {"tokens": NP * LP, "ms": t * 1e3, "tokens_per_s": NP * LP / t}}
+    for i in range(B):
+        eng.cache.admit(("d", i)); eng.cache.reserve(("d", i), CTX + 1)
+    db = StepBatch.build([(eng.cache.seqs[("d", i)].slot, CTX, 5, [int(torch.randint(0, V, (1,), generator=g))]) for i in range(B)],
+                         eng.cache.sync_block_table(), dev)
+    t = time_kernel(lambda: (model.logits(model.forward(db, eng.cache)), 1)[1], reps * 4, stream)
+    rec["decode"] = {"batch": B, "ctx": CTX, "ms": t * 1e3, "tokens_per_s": B / t}
+    return rec, pb, db
+
+
+def hybrid_mixer_times(mixer, run_cache, pb, db, T, reps, stream):
+    """Seconds of one mixer (without its projections) on the prompt batch and on the decode batch."""
+    import torch
+
+    B, dev = HYBRID_LOAD[0], mixer.w_out.device
+    raw = lambda: torch._C._cuda_getCurrentRawStream(0)
+    proj = torch.randn(T, mixer.in_features, device=dev).to(torch.bfloat16)
+    cat = torch.empty(T, mixer.out_features, dtype=torch.bfloat16, device=dev)
+    scratch = torch.empty(max(1, mixer.scratch_floats(T)), dtype=torch.float32, device=dev)
+    tp = time_kernel(lambda: (mixer.run(proj, cat, pb, run_cache, 64, scratch, 0, raw()), 1)[1], reps, stream)
+    td = time_kernel(lambda: (mixer.run(proj[:B], cat[:B], db, run_cache, 64, scratch, 0, raw()), 1)[1], reps * 4, stream)
+    return tp, td
+
+
+def hybrid_lone_mixer(mcfg, W, seed, dev):
+    """A mixer of another design with random weights."""
+    import torch
+
+    from qserve_b200.hybrid import MIXERS, random_weights
+    from qserve_b200.modelcfg import HybridConfig, HybridLayerConfig
+
+    c1 = HybridConfig("bench", 8, W, 1e-5, (HybridLayerConfig("m", mcfg, None),))
+    w = {k[len("l0.mix."):]: v for k, v in random_weights(c1, seed, dev).items() if k.startswith("l0.mix.")}
+    return MIXERS[type(mcfg)](mcfg, w, 1e-5, torch.bfloat16, dev)
+
+
+# ------------------------------------------------------------------------------------------------------------
 # --zuzezen: the Zuzezen decoder beside the closest existing model (the Rizurax hybrid decoder) at equal size
 # ------------------------------------------------------------------------------------------------------------
 def zuzezen_block(args):
@@ -1166,39 +1226,13 @@ def zuzezen_block(args):
     stream = torch.cuda.current_stream()
     reps = max(3, args.kernel_reps)
     raw = lambda: torch._C._cuda_getCurrentRawStream(0)
-    B, CTX, NP, LP, KR, R, WIN, KEEP = 64, 1024, 4, 2048, 512, 64, 1024, 4
+    (B, CTX, NP, LP), KR, R, WIN, KEEP = HYBRID_LOAD, 512, 64, 1024, 4
     out = {"metric": "Zuzezen decoder throughput (tokens/s, random weights, bf16, 5 layers)", "unit": "tokens/s", "impl": "ours",
            "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops}, "sizes": {}}
 
-    def steps(model, eng, V, g):
-        prompts = [torch.randint(0, V, (LP,), generator=g).tolist() for _ in range(NP)]
-        for i, p_ in enumerate(prompts):
-            eng.cache.admit(("p", i)); eng.cache.reserve(("p", i), LP)
-        pb = StepBatch.build([(eng.cache.seqs[("p", i)].slot, 0, -1, p_) for i, p_ in enumerate(prompts)], eng.cache.sync_block_table(), dev,
-                             eng.cache.page_size)
-        t = time_kernel(lambda: (model.forward(pb, eng.cache), 1)[1], reps, stream)
-        rec = {"prefill": {"tokens": NP * LP, "ms": t * 1e3, "tokens_per_s": NP * LP / t}}
-        for i in range(B):
-            eng.cache.admit(("d", i)); eng.cache.reserve(("d", i), CTX + 1)
-        db = StepBatch.build([(eng.cache.seqs[("d", i)].slot, CTX, 5, [int(torch.randint(0, V, (1,), generator=g))]) for i in range(B)],
-                             eng.cache.sync_block_table(), dev)
-        t = time_kernel(lambda: (model.logits(model.forward(db, eng.cache)), 1)[1], reps * 4, stream)
-        rec["decode"] = {"batch": B, "ctx": CTX, "ms": t * 1e3, "tokens_per_s": B / t}
-        return rec, pb, db
-
-    def mixer_times(mixer, run_cache, pb, db, T):
-        proj = torch.randn(T, mixer.in_features, device=dev).to(torch.bfloat16)
-        cat = torch.empty(T, mixer.out_features, dtype=torch.bfloat16, device=dev)
-        scratch = torch.empty(max(1, mixer.scratch_floats(T)), dtype=torch.float32, device=dev)
-        tp = time_kernel(lambda: (mixer.run(proj, cat, pb, run_cache, 64, scratch, 0, raw()), 1)[1], reps, stream)
-        td = time_kernel(lambda: (mixer.run(proj[:B], cat[:B], db, run_cache, 64, scratch, 0, raw()), 1)[1], reps * 4, stream)
-        return tp, td
-
-    def lone_mixer(mcfg, W, seed):
-        """A mixer of another design with random weights, and storage for it in a cache of its own."""
-        c1 = HybridConfig("bench", 8, W, 1e-5, (HybridLayerConfig("m", mcfg, None),))
-        w = {k[len("l0.mix."):]: v for k, v in random_weights(c1, seed, dev).items() if k.startswith("l0.mix.")}
-        return MIXERS[type(mcfg)](mcfg, w, 1e-5, torch.bfloat16, dev)
+    steps = lambda model, eng, V, g: hybrid_steps(model, eng, V, g, reps, stream)
+    mixer_times = lambda mixer, run_cache, pb, db, T: hybrid_mixer_times(mixer, run_cache, pb, db, T, reps, stream)
+    lone_mixer = lambda mcfg, W, seed: hybrid_lone_mixer(mcfg, W, seed, dev)
 
     for name, (W, H, G, D, FF, V) in HYBRID_SIZES.items():
         T = NP * LP
@@ -1306,6 +1340,127 @@ def zuzezen_block(args):
 
 
 # ------------------------------------------------------------------------------------------------------------
+# --nagosun: the Nagosun decoder beside the closest existing model (the Zuzezen decoder's attention layers) at equal size
+# ------------------------------------------------------------------------------------------------------------
+def nagosun_block(args):
+    """Prefill and decode (HYBRID_LOAD) of a five-layer Nagosun stack latent attention | attention | attention | latent attention | attention,
+    a feed-forward in every layer, beside a Zuzezen stack of the same layout, width, head geometry, feed-forward size and window; then
+    each Nagosun kernel beside the like kernel of Zuzezen on the same batches: windowed attention with capped scores, unit-RMS values, a
+    spare softmax term and a gate per output number beside the one with tied values, kept positions and a gate per head; latent
+    attention under a window and without one beside the one with a sink and a wide gate; the landing kernel (bias, gate, grouped norm,
+    residual, grouped norm) beside the post-norm landing kernel; the silu gate beside the biased one."""
+    import torch
+
+    from qserve_b200._lib import check, lib
+    from qserve_b200.engine import Engine
+    from qserve_b200.hybrid import HybridDecoder, random_weights
+    from qserve_b200.modelcfg import AttentionMixerConfig, HybridConfig, HybridLayerConfig, LatentAttentionMixerConfig, MlpConfig, RotaryConfig
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm_gbs = peaks()[0]
+    try:
+        tflops = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"]
+    except (OSError, KeyError, ValueError):
+        tflops = 1590.0
+    stream = torch.cuda.current_stream()
+    reps = max(3, args.kernel_reps)
+    raw = lambda: torch._C._cuda_getCurrentRawStream(0)
+    (B, CTX, NP, LP), KR, R, WIN, KEEP, GROUPS = HYBRID_LOAD, 512, 64, 1024, 4, 4
+    T = NP * LP
+    out = {"metric": "Nagosun decoder throughput (tokens/s, random weights, bf16, 5 layers)", "unit": "tokens/s", "impl": "ours", "dtype": "bf16",
+           "data": "synthetic", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops}, "load": {"decode_batch": B, "ctx": CTX, "prompts": NP, "prompt": LP,
+                                                                                              "window": WIN}, "sizes": {}}
+    pairs_all = NP * (LP * (LP + 1) // 2)
+    pairs_win = NP * sum(min(i + 1, WIN) for i in range(LP))
+    pairs_kept = pairs_win + NP * sum(min(KEEP, i + 1 - WIN) for i in range(WIN, LP))
+    seen = min(CTX + 1, WIN)
+
+    def attention_rec(tp, td, H, G, D, pairs, keys):
+        return {"prefill_us": tp * 1e6, "prefill_tflops": H * pairs * 4 * D / tp / 1e12, "prefill_frac_of_measured_bf16_peak": H * pairs * 4 * D / tp / 1e12 / tflops,
+                "decode_us": td * 1e6, "decode_frac_of_measured_hbm": B * keys * G * 2 * D * 2 / td / 1e9 / hbm_gbs}
+
+    def latent_rec(tp, td, H, D, pairs, keys):
+        useful = H * pairs * 2 * (D + R + D)
+        return {"prefill_us": tp * 1e6, "prefill_tflops": useful / tp / 1e12, "prefill_frac_of_measured_bf16_peak": useful / tp / 1e12 / tflops,
+                "decode_us": td * 1e6, "decode_frac_of_measured_hbm": B * keys * (KR + R) * 2 / td / 1e9 / hbm_gbs}
+
+    for name, (W, H, G, D, FF, V) in HYBRID_SIZES.items():
+        lat = LatentAttentionMixerConfig(H, D, R, D, KR, 0, RotaryConfig(R, 1e6), (D + R) ** -0.5, gate=False, window=WIN)
+        att = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, window=WIN, distance_slope=8.0, gate_wide=True, softcap=50.0, value_norm=True,
+                                   sink_score=0.0, out_bias=True)
+        ffc = MlpConfig("dense", FF, act="silu")
+        cfg = HybridConfig("Nagosun", V, W, 1e-6, tuple(HybridLayerConfig("latent_attention" if m is lat else "attention", m, ffc) for m in (lat, att, att, lat, att)),
+                           norm_offset=0.0, block="sandwich", norm_groups=GROUPS, residual_mult=0.5, residual_gate=True, embed_norm=True, logit_scale=0.25)
+        zlat = LatentAttentionMixerConfig(H, D, R, D, KR, 0, RotaryConfig(R, 1e6, 4.0, 4096, 32.0, 1.0), (D + R) ** -0.5, gate=True, gate_wide=True, sink=True)
+        zatt = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, qk_norm=True, window=WIN, keep_first=KEEP, qk_gain=True, tied_values=True,
+                                    distance_slope=8.0, head_gate=True)
+        zffc = MlpConfig("dense", FF, gated=True, bias=True, act="silu")
+        zcfg = HybridConfig("Zuzezen", V, W, 1e-5, tuple(HybridLayerConfig("latent_attention" if m is zlat else "attention", m, zffc)
+                                                        for m in (zlat, zatt, zatt, zlat, zatt)), norm_offset=1.0, block="post", embed_scale=8.0, layer_scale=True)
+        g = torch.Generator().manual_seed(0)
+        kern, like = {}, {}
+        with torch.no_grad():
+            model = HybridDecoder(cfg, random_weights(cfg, 0, dev), torch.bfloat16, dev)
+            eng = Engine(model, max_tokens=B * (CTX + 64) + NP * LP, max_seqs=B + NP)
+            rec, pb, db = hybrid_steps(model, eng, V, g, reps, stream)
+            times = lambda mixer, store: hybrid_mixer_times(mixer, store, pb, db, T, reps, stream)
+            kern["attention(bias+unit-RMS values+append, tiles / head groups with window, capped scores, distance bias, spare term, wide gate)"] = \
+                attention_rec(*times(model.layers[1].mixer, eng.cache.runs[1]), H, G, D, pairs_win, seen)
+            kern["latent_attention(norm+rotate+append+keys and values of every head or latent tiles, window)"] = \
+                latent_rec(*times(model.layers[0].mixer, eng.cache.runs[0]), H, D, pairs_win, seen)
+            for key, mc in (("attention(without the score cap)", dict(softcap=0.0)), ("attention(without a window)", dict(window=0))):
+                lone = hybrid_lone_mixer(dataclasses.replace(att, **mc), W, 1, dev)
+                kern[key] = attention_rec(*times(lone, eng.cache.mixer_storage(lone.m)), H, G, D, pairs_all if mc.get("window") == 0 else pairs_win,
+                                          CTX + 1 if mc.get("window") == 0 else seen)
+            lone = hybrid_lone_mixer(dataclasses.replace(lat, window=0), W, 1, dev)
+            kern["latent_attention(without a window)"] = latent_rec(*times(lone, eng.cache.mixer_storage(lone.m)), H, D, pairs_all, CTX + 1)
+            lone = hybrid_lone_mixer(zatt, W, 1, dev)
+            like["attention(bias+unit RMS+gains+append, window with kept positions, distance bias, head gate)"] = \
+                attention_rec(*times(lone, eng.cache.mixer_storage(lone.m)), H, G, D, pairs_kept, seen + (KEEP if CTX + 1 > WIN else 0))
+            lone = hybrid_lone_mixer(zlat, W, 1, dev)
+            like["latent_attention(sink, wide gate, no window)"] = latent_rec(*times(lone, eng.cache.mixer_storage(lone.m)), H, D, pairs_all, CTX + 1)
+            del lone
+            ly = model.layers[1]
+            x, y = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+            h1 = torch.empty(T, W, dtype=torch.bfloat16, device=dev)
+            gates = torch.randn(T, ly.w_mix_in.shape[0], device=dev).to(torch.bfloat16)   # rows of the stacked product the gate's columns lie in
+            gate = gates[:, ly.gate1:]
+            tn = time_kernel(lambda: (check(lib.qs_hyb_gated_norm_update(h1.data_ptr(), x.data_ptr(), 0, y.data_ptr(), 1, ly.mixer.out_bias.data_ptr(), gate.data_ptr(),
+                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.5, ly.norm2.data_ptr(),
+                                                                         GROUPS, 0.0, 1e-6, T, W, 0, raw())), 1)[1], reps, stream)
+            kern["gated_norm_update(fp32 rows in, bias, gate, grouped norm, residual, grouped norm of the stream)"] = {
+                "us": tn * 1e6, "frac_of_measured_hbm": T * W * 16 / tn / 1e9 / hbm_gbs}
+            tn = time_kernel(lambda: (check(lib.qs_hyb_gated_norm_update(h1.data_ptr(), x.data_ptr(), 0, y.data_ptr(), 1, ly.mixer.out_bias.data_ptr(), gate.data_ptr(),
+                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.5, ly.norm2.data_ptr(),
+                                                                         GROUPS, 0.0, 1e-6, B, W, 0, raw())), 1)[1], reps * 4, stream)
+            kern["gated_norm_update, decode batch"] = {"us": tn * 1e6}
+            w1 = torch.ones(W, device=dev)
+            tn = time_kernel(lambda: (check(lib.qs_hyb_post_norm_update(h1.data_ptr(), x.data_ptr(), y.data_ptr(), 1, w1.data_ptr(), w1.data_ptr(), w1.data_ptr(), 1.0, 1e-5,
+                                                                        T, W, 0, raw())), 1)[1], reps, stream)
+            like["post_norm_update(fp32 rows in, bias, norm, layer scale, residual, bf16 copy)"] = {"us": tn * 1e6, "frac_of_measured_hbm": T * W * 14 / tn / 1e9 / hbm_gbs}
+            tn = time_kernel(lambda: (check(lib.qs_hyb_post_norm_update(h1.data_ptr(), x.data_ptr(), y.data_ptr(), 1, w1.data_ptr(), w1.data_ptr(), w1.data_ptr(), 1.0, 1e-5,
+                                                                        B, W, 0, raw())), 1)[1], reps * 4, stream)
+            like["post_norm_update, decode batch"] = {"us": tn * 1e6}
+            gu = torch.randn(T, ly.w_ff_in.shape[0], device=dev).to(torch.bfloat16)
+            act, fb = torch.empty(T, FF, dtype=torch.bfloat16, device=dev), torch.zeros(2 * FF, device=dev)
+            tg = time_kernel(lambda: (check(lib.qs_hyb_bias_gated_act(act.data_ptr(), FF, gu.data_ptr(), gu.stride(0), None, T, FF, 1, 0, raw())), 1)[1], reps, stream)
+            kern["silu_mul(rows with the gate's columns beside)"] = {"us": tg * 1e6, "frac_of_measured_hbm": T * FF * 6 / tg / 1e9 / hbm_gbs}
+            tg = time_kernel(lambda: (check(lib.qs_hyb_bias_gated_act(act.data_ptr(), FF, gu.data_ptr(), 2 * FF, fb.data_ptr(), T, FF, 1, 0, raw())), 1)[1], reps, stream)
+            like["bias_silu_mul"] = {"us": tg * 1e6, "frac_of_measured_hbm": T * FF * 6 / tg / 1e9 / hbm_gbs}
+            del eng, model, x, y, h1, gates, gate, gu, act
+            torch.cuda.empty_cache()
+            model = HybridDecoder(zcfg, random_weights(zcfg, 0, dev), torch.bfloat16, dev)
+            eng = Engine(model, max_tokens=B * (CTX + 64) + NP * LP, max_seqs=B + NP)
+            peer, _, _ = hybrid_steps(model, eng, V, g, reps, stream)
+            del eng, model
+        torch.cuda.empty_cache()
+        rec["kernels"], rec["like_kernels_of_zuzezen"], rec["zuzezen_equal_size"] = kern, like, peer
+        out["sizes"][name] = rec
+    print(json.dumps(out), flush=True)
+
+
+# ------------------------------------------------------------------------------------------------------------
 def main():
     args = parse()
     rank = int(os.environ.get("RANK", "0"))
@@ -1329,6 +1484,10 @@ def main():
     if args.zuzezen:
         if rank == 0:
             zuzezen_block(args)
+        return
+    if args.nagosun:
+        if rank == 0:
+            nagosun_block(args)
         return
     if args.impl == "reference-gpu":
         if rank == 0:
