@@ -1366,7 +1366,7 @@ def nagosun_block(args):
     stream = torch.cuda.current_stream()
     reps = max(3, args.kernel_reps)
     raw = lambda: torch._C._cuda_getCurrentRawStream(0)
-    (B, CTX, NP, LP), KR, R, WIN, KEEP, GROUPS = HYBRID_LOAD, 512, 64, 1024, 4, 4
+    (B, CTX, NP, LP), KR, R, WIN, KEEP, GROUPS = HYBRID_LOAD, 512, 64, 1024, 4, 8
     T = NP * LP
     out = {"metric": "Nagosun decoder throughput (tokens/s, random weights, bf16, 5 layers)", "unit": "tokens/s", "impl": "ours", "dtype": "bf16",
            "data": "synthetic", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops}, "load": {"decode_batch": B, "ctx": CTX, "prompts": NP, "prompt": LP,
@@ -1387,11 +1387,11 @@ def nagosun_block(args):
 
     for name, (W, H, G, D, FF, V) in HYBRID_SIZES.items():
         lat = LatentAttentionMixerConfig(H, D, R, D, KR, 0, RotaryConfig(R, 1e6), (D + R) ** -0.5, gate=False, window=WIN)
-        att = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, window=WIN, distance_slope=8.0, gate_wide=True, softcap=50.0, value_norm=True,
+        att = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, window=WIN, distance_slope=8.0, gate_wide=True, softcap=30.0, value_norm=True,
                                    sink_score=0.0, out_bias=True)
         ffc = MlpConfig("dense", FF, act="silu")
-        cfg = HybridConfig("Nagosun", V, W, 1e-6, tuple(HybridLayerConfig("latent_attention" if m is lat else "attention", m, ffc) for m in (lat, att, att, lat, att)),
-                           norm_offset=0.0, block="sandwich", norm_groups=GROUPS, residual_mult=0.5, residual_gate=True, embed_norm=True, logit_scale=0.25)
+        cfg = HybridConfig("Nagosun", V, W, 1e-5, tuple(HybridLayerConfig("latent_attention" if m is lat else "attention", m, ffc) for m in (lat, att, att, lat, att)),
+                           norm_offset=0.0, block="sandwich", norm_groups=GROUPS, residual_mult=0.7, residual_gate=True, embed_norm=True, logit_scale=2.0)
         zlat = LatentAttentionMixerConfig(H, D, R, D, KR, 0, RotaryConfig(R, 1e6, 4.0, 4096, 32.0, 1.0), (D + R) ** -0.5, gate=True, gate_wide=True, sink=True)
         zatt = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, qk_norm=True, window=WIN, keep_first=KEEP, qk_gain=True, tied_values=True,
                                     distance_slope=8.0, head_gate=True)
@@ -1427,13 +1427,13 @@ def nagosun_block(args):
             gates = torch.randn(T, ly.w_mix_in.shape[0], device=dev).to(torch.bfloat16)   # rows of the stacked product the gate's columns lie in
             gate = gates[:, ly.gate1:]
             tn = time_kernel(lambda: (check(lib.qs_hyb_gated_norm_update(h1.data_ptr(), x.data_ptr(), 0, y.data_ptr(), 1, ly.mixer.out_bias.data_ptr(), gate.data_ptr(),
-                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.5, ly.norm2.data_ptr(),
-                                                                         GROUPS, 0.0, 1e-6, T, W, 0, raw())), 1)[1], reps, stream)
+                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.7, ly.norm2.data_ptr(),
+                                                                         GROUPS, 0.0, 1e-5, T, W, 0, raw())), 1)[1], reps, stream)
             kern["gated_norm_update(fp32 rows in, bias, gate, grouped norm, residual, grouped norm of the stream)"] = {
                 "us": tn * 1e6, "frac_of_measured_hbm": T * W * 16 / tn / 1e9 / hbm_gbs}
             tn = time_kernel(lambda: (check(lib.qs_hyb_gated_norm_update(h1.data_ptr(), x.data_ptr(), 0, y.data_ptr(), 1, ly.mixer.out_bias.data_ptr(), gate.data_ptr(),
-                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.5, ly.norm2.data_ptr(),
-                                                                         GROUPS, 0.0, 1e-6, B, W, 0, raw())), 1)[1], reps * 4, stream)
+                                                                         gate.stride(0), ly.gate1_b.data_ptr(), ly.norm1_back.data_ptr(), 0.7, ly.norm2.data_ptr(),
+                                                                         GROUPS, 0.0, 1e-5, B, W, 0, raw())), 1)[1], reps * 4, stream)
             kern["gated_norm_update, decode batch"] = {"us": tn * 1e6}
             w1 = torch.ones(W, device=dev)
             tn = time_kernel(lambda: (check(lib.qs_hyb_post_norm_update(h1.data_ptr(), x.data_ptr(), y.data_ptr(), 1, w1.data_ptr(), w1.data_ptr(), w1.data_ptr(), 1.0, 1e-5,
