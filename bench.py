@@ -887,7 +887,7 @@ def toderax_block(args):
                     "weights_frac_of_measured_hbm": 3 * W * (min(E, n * TOP) * moe.ff + moe.shared_ff) * 2 / tm / 1e9 / hbm_gbs}
             route, ti, tw = torch.empty(T, E, device=dev), torch.empty(T, TOP, dtype=torch.int32, device=dev), torch.empty(T, TOP, device=dev)
             tr = time_kernel(lambda: (check(lib.qs_hyb_moe_router(route.data_ptr(), ti.data_ptr(), tw.data_ptr(), h.data_ptr(), ly_g.ff.w_router.data_ptr(),
-                                                                  T, W, E, TOP, 0, None, 1, 1, 0, raw())), 1)[1], reps, stream)
+                                                                  T, W, E, TOP, 0, None, 1, 1, 1, 1.0, 0, raw())), 1)[1], reps, stream)
             kern["moe_router"] = {"us": tr * 1e6, "frac_of_measured_hbm": T * W * 2 / tr / 1e9 / hbm_gbs}
             gu = torch.randn(T * TOP, 2 * moe.ff, device=dev).to(torch.bfloat16)
             act = torch.empty(T * TOP, moe.ff, dtype=torch.bfloat16, device=dev)
@@ -1098,7 +1098,7 @@ def nusuvik_block(args):
             route, ti, tw = torch.empty(T, E, device=dev), torch.empty(T, TOP, dtype=torch.int32, device=dev), torch.empty(T, TOP, device=dev)
             for mode, label in ((1, "router_sigmoid_groups"), (0, "router_softmax(the other design's)")):
                 tr = time_kernel(lambda: (check(lib.qs_hyb_moe_router(route.data_ptr(), ti.data_ptr(), tw.data_ptr(), h.data_ptr(), ff1.w_router.data_ptr(),
-                                                                      T, W, E, TOP, mode, ff1.correction.data_ptr(), 4, 2, 0, raw())), 1)[1], reps, stream)
+                                                                      T, W, E, TOP, mode, ff1.correction.data_ptr(), 4, 2, 1, 1.0, 0, raw())), 1)[1], reps, stream)
                 kern[label] = {"us": tr * 1e6, "frac_of_measured_hbm": T * W * 2 / tr / 1e9 / hbm_gbs}
             # the like feed-forward of the closest design with experts: softmax router, clamped activation, no shared expert, equal sizes
             tmoe = MoeConfig(E, TOP, FF // TOP, 7.0)

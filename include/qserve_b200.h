@@ -301,6 +301,38 @@ QS_API int qs_hyb_qk_prepare_append(void* proj, int64_t stride, const float* bia
                                     const float* inv_freq, int rot_layout, int rot_dims, int unit_rms, float eps, int tokens_n, int heads,
                                     int kv_heads, int dim, int vdim, int page_size, const float* q_gain, const float* k_gain, int tied_values,
                                     int value_rms, int dtype, void* stream);
+/* Query / key preparation where q and k are each normed as one row ahead of the split into heads: rows [q_cols q | k_cols k | v_cols v], bias
+ * (fp32, same layout) may be NULL; q *= rsqrt(mean(q^2) + eps) q_gain f, k *= rsqrt(mean(k^2) + eps) k_gain (fp32 gains over the rows),
+ * f = 1 + temp_coef ln(floor((position + 1) / temp_every) + 1); q in place, k and v (+ bias) to the pages [page][page_size][cols]. */
+QS_API int qs_hyb_qk_row_norm_append(void* proj, int64_t stride, const float* bias, const float* q_gain, const float* k_gain, float temp_coef,
+                                     float temp_every, const int32_t* tok_slot, const int32_t* tok_pos, const int32_t* block_table, int max_blocks,
+                                     void* kpool, void* vpool, float eps, int tokens_n, int q_cols, int k_cols, int v_cols, int page_size, int dtype,
+                                     void* stream);
+/* State space layer (csrc/hybrid_recurrent.cu) over projection rows [inner z | inner x | G*N B | G*N C | H dt], inner = H vdim, N = state_n: x, B, C pass
+ * a causal convolution of `taps` inputs per channel (conv_w fp32 [channels, taps], the last column for the current token; conv_b fp32, may be
+ * NULL) and silu; dt <- softplus(dt + dt_bias); per head (head h reads group h / (H / G)) S <- exp(-exp(a_log) dt) S + dt B x^T,
+ * y = S^T C + skip x; out = rms(y silu(z)) norm_w out_scale with the RMS over norm_groups equal parts of the row.  state fp32
+ * [slots, H, N, vdim], conv_state fp32 [slots, taps - 1, channels]; a run that starts at position 0 starts from zero.  prep fp32
+ * [tokens, qs_hyb_state_space_prep_floats] and o_raw fp32 [tokens, inner] are scratch. */
+QS_API int qs_hyb_state_space_prep_floats(int heads, int groups, int state_n, int vdim);
+QS_API int qs_hyb_state_space(void* out, int64_t out_stride, float* prep, float* o_raw, const void* proj, int64_t stride, const float* conv_w,
+                              const float* conv_b, float* conv_state, float* state, const float* a_log, const float* dt_bias, const float* skip,
+                              const float* norm_w, int norm_groups, float out_scale, const int32_t* tok_entry, const int32_t* tok_pos,
+                              const int32_t* entry_start, const int32_t* entry_len, const int32_t* entry_slot, const int32_t* entry_pos0, int tokens_n,
+                              int entries, int heads, int groups, int state_n, int vdim, int taps, float eps, int dtype, void* stream);
+/* Gated linear recurrent unit over projection rows [width y | width x].  qs_hyb_lru_conv: u = causal convolution of x + x_bias (conv_w, conv_b as
+ * above), storage type [tokens, width].  qs_hyb_lru_scan: with the gate logits z fp32 [blocks, tokens, 2 width / blocks] (r's, then i's),
+ * log a = rate sigmoid(z_r + r_bias) (rate fp32 [width], negative), S <- a S + sqrt(1 - a^2) sigmoid(z_i + i_bias) u, out = S gelu_tanh(y + y_bias).
+ * state fp32 [slots, width].  Entries of at least long_min tokens are the ones that the tiles (of tile_rows rows) cover; n_short: tokens of the
+ * others; sums fp32 [n_tiles, 2, width] is scratch. */
+QS_API int qs_hyb_lru_conv(void* u, const void* proj, int64_t stride, const float* x_bias, const float* conv_w, const float* conv_b, float* conv_state,
+                           const int32_t* tok_entry, const int32_t* tok_pos, const int32_t* entry_start, const int32_t* entry_len,
+                           const int32_t* entry_slot, const int32_t* entry_pos0, int tokens_n, int entries, int width, int taps, int dtype, void* stream);
+QS_API int qs_hyb_lru_scan(void* out, int64_t out_stride, float* state, float* sums, const void* u, const float* z, const void* proj, int64_t stride,
+                           const float* y_bias, const float* r_bias, const float* i_bias, const float* rate, const int32_t* tile_entry,
+                           const int32_t* tile_row0, int n_tiles, int n_short, const int32_t* entry_start, const int32_t* entry_len,
+                           const int32_t* entry_slot, const int32_t* entry_pos0, int tokens_n, int entries, int width, int blocks, int tile_rows,
+                           int long_min, int dtype, void* stream);
 /* Gate recurrence (HGRN2) over projection rows [H*dim q | H*dim f | H*vdim v]: q <- silu(q), f <- lower + (1 - lower) sigmoid(f + f_bias)
  * (fp32 [H*dim] each), per head S <- diag(f) S + (1 - f) v^T, o = S^T q, out = o rsqrt(mean(o^2) + eps) norm_w (fp32 [vdim], may be NULL).
  * state fp32 [slots, H, dim, vdim]; a run that starts at position 0 starts from zero.  prep fp32 [tokens, 2 H dim + H vdim] and o_raw fp32
@@ -329,11 +361,13 @@ QS_API int qs_hyb_gated_linear(void* out, int64_t out_stride, float* prep, float
  * QS_ROUTER_SOFTMAX: scores softmax(z) over all experts, the `top` largest kept as they are (correction, groups, keep unused).
  * QS_ROUTER_SIGMOID_GROUPS: scores s = sigmoid(z); the choice is made on s + correction (fp32 [experts], may be NULL): the experts form
  * `groups` equal runs of neighbours, a group's score is the sum of its two largest choice scores, only experts of the `keep` best groups can
- * be chosen, the `top` largest choice scores win; weights s / (sum of the winners' s + 1e-20). */
+ * be chosen, the `top` largest choice scores win; weights s / (sum of the winners' s + 1e-20), or s as it is (renormalize = 0).
+ * weight_scale: a factor on every weight. */
 #define QS_ROUTER_SOFTMAX 0
 #define QS_ROUTER_SIGMOID_GROUPS 1
 QS_API int qs_hyb_moe_router(float* route, int32_t* top_idx, float* top_w, const void* h, const float* w_router, int tokens_n, int width,
-                             int experts, int top, int mode, const float* correction, int groups, int keep, int dtype, void* stream);
+                             int experts, int top, int mode, const float* correction, int groups, int keep, int renormalize, float weight_scale,
+                             int dtype, void* stream);
 /* Activation of all experts' columns of a token: in rows [F gate | F up], F = experts * ff + ff_shared (the shared expert's columns last);
  * g = min(gate, limit), u = clamp(up, -limit, limit), out = route[t, expert] g sigmoid(alpha g) (u + shift); shared columns: weight 1 and
  * limit_shared.  limit = +inf, alpha = 1, shift = 0 is silu(gate) * up.  out [tokens, F]. */
@@ -362,6 +396,9 @@ QS_API int qs_hyb_stream_update_norm(void* out_h, void* cat_out, float* x, const
 /* out[t, i] = gelu_tanh(in[t, i] + bias[i]) (bias fp32, may be NULL); rows of in_stride / out_stride elements */
 QS_API int qs_hyb_bias_gelu_tanh(void* out, int64_t out_stride, const void* in, int64_t in_stride, const float* bias, int tokens_n, int ff,
                                  int dtype, void* stream);
+/* out[t, i] = max(in[t, i] + bias[i], 0)^2 (bias fp32, may be NULL); rows of in_stride / out_stride elements */
+QS_API int qs_hyb_bias_relu_squared(void* out, int64_t out_stride, const void* in, int64_t in_stride, const float* bias, int tokens_n, int ff,
+                                    int dtype, void* stream);
 /* Post-norm residual update: y = add (+ add_bias, fp32 [width], may be NULL); x <- x + y rsqrt(mean(y^2) + eps) (offset + w) (* ls, fp32
  * [width], may be NULL); out_h (may be NULL) <- x in the storage type.  add rows: fp32 if add_f32, else storage type; x fp32 [tokens, width]. */
 QS_API int qs_hyb_post_norm_update(void* out_h, float* x, const void* add, int add_f32, const float* add_bias, const float* w, const float* ls,

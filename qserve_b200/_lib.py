@@ -73,7 +73,15 @@ SIGNATURES = {
     "qs_hyb_bias_gated_act": (c_int, [_P, _L, _P, _L, _P, _I, _I, _I, _I, _P]),
     "qs_hyb_gate_recurrence": (c_int, [_P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P]),
     "qs_hyb_retention": (c_int, [_P, _L, _P, _P, _P, _L, _P, _P, _I, _F, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P]),
-    "qs_hyb_moe_router": (c_int, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _P]),
+    "qs_hyb_moe_router": (c_int, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _I, _P]),
+    "qs_hyb_qk_row_norm_append": (c_int, [_P, _L, _P, _P, _P, _F, _F, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P]),
+    "qs_hyb_bias_relu_squared": (c_int, [_P, _L, _P, _L, _P, _I, _I, _I, _P]),
+    # csrc/hybrid_recurrent.cu
+    "qs_hyb_state_space_prep_floats": (c_int, [_I, _I, _I, _I]),
+    "qs_hyb_state_space": (c_int, [_P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
+                                   _P]),
+    "qs_hyb_lru_conv": (c_int, [_P, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P]),
+    "qs_hyb_lru_scan": (c_int, [_P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P]),
     "qs_hyb_moe_act": (c_int, [_P, _P, _P, _I, _I, _I, _F, _I, _F, _F, _F, _I, _P]),
     "qs_hyb_moe_plan": (c_int, [_P, _P, _P, _P, _P, _I, _I, _I, _P]),
     "qs_hyb_moe_plan_work_ints": (_L, [_I]),

@@ -3,8 +3,8 @@ state slots (one per live sequence) for what a recurrent layer carries from toke
 
 * Pages hold `page_size` positions.  A sequence owns a list of pages (its block-table row); page ids are valid in every attention layer
   run's K and V pool, as in the reference's block manager (qserve/core/block_manager.py: one block table per sequence, all layers).
-* A slot holds, per recurrent layer run, the fp32 state (and, for the delta rule, the convolution's last inputs); the slot index is also the
-  block-table row.  Two mixers side by side keep their storage side by side ("left" / "right").
+* A slot holds, per recurrent layer run, the fp32 state (and, for layers with short convolutions, the convolution's last inputs); the slot index
+  is also the block-table row.  Two mixers side by side keep their storage side by side ("left" / "right").
 * Released pages and slots go back to LIFO free lists and are handed out again first: nothing is cleared on release, a recurrent layer
   starts a sequence (position 0) from zero by itself and attention never reads beyond a sequence's own length.
 """
@@ -15,8 +15,8 @@ from typing import Dict, List
 
 import torch
 
-from .modelcfg import (AttentionMixerConfig, DeltaMixerConfig, GatedLinearMixerConfig, GateRecurrenceMixerConfig, HybridConfig,
-                       LatentAttentionMixerConfig, ParallelMixerConfig, RetentionMixerConfig)
+from .modelcfg import (AttentionMixerConfig, DeltaMixerConfig, GatedLinearMixerConfig, GatedUnitMixerConfig, GateRecurrenceMixerConfig,
+                       HybridConfig, LatentAttentionMixerConfig, ParallelMixerConfig, RetentionMixerConfig, StateSpaceMixerConfig)
 
 
 class OutOfPages(RuntimeError):
@@ -84,6 +84,13 @@ class HybridCache:
                     "conv": torch.zeros((max_seqs, max(m.conv - 1, 1), c), dtype=torch.float32, device=device)}
         if isinstance(m, (GateRecurrenceMixerConfig, RetentionMixerConfig, GatedLinearMixerConfig)):
             return {"state": torch.zeros((max_seqs, m.heads, m.dim, m.vdim), dtype=torch.float32, device=device)}
+        if isinstance(m, StateSpaceMixerConfig):
+            c = m.heads * m.vdim + 2 * m.groups * m.state
+            return {"state": torch.zeros((max_seqs, m.heads, m.state, m.vdim), dtype=torch.float32, device=device),
+                    "conv": torch.zeros((max_seqs, max(m.conv - 1, 1), c), dtype=torch.float32, device=device)}
+        if isinstance(m, GatedUnitMixerConfig):
+            return {"state": torch.zeros((max_seqs, m.width), dtype=torch.float32, device=device),
+                    "conv": torch.zeros((max_seqs, max(m.conv - 1, 1), m.width), dtype=torch.float32, device=device)}
         if isinstance(m, ParallelMixerConfig):
             return {"left": self.mixer_storage(m.left), "right": self.mixer_storage(m.right)}
         raise TypeError(type(m))

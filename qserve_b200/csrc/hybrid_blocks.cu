@@ -300,6 +300,87 @@ __global__ void qk_prepare_append_kernel(ST* __restrict__ proj, long long stride
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------------
+// Query / key preparation where q and k are each normed as one row, ahead of the split into heads, and the append to the paged cache:
+//   projection row [NQ q | NK k | NV v] (+ bias);  q <- q rsqrt(mean(q^2) + eps) q_gain f,  k <- k rsqrt(mean(k^2) + eps) k_gain,  with the query
+//   factor f = 1 + temp_coef ln(floor((position + 1) / temp_every) + 1)  (temp_coef 0: none)
+// grid (tokens, 3): the blocks of a token finish q in place, store k, store v.  K pages [page][page_size][NK], V pages [page][page_size][NV].
+// ---------------------------------------------------------------------------------------------------------------------------------
+template <typename ST, int V>
+__device__ __forceinline__ void load_biased(float (&x)[V], const ST* p, const float* bias, int i) {
+  if constexpr (V == 4) {
+    const float4 q = ld4(p + i);
+    x[0] = q.x; x[1] = q.y; x[2] = q.z; x[3] = q.w;
+  } else {
+    x[0] = ldf(p + i);
+  }
+  if (bias != nullptr) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[v] += bias[i + v];
+  }
+}
+
+template <typename ST, int V>
+__global__ void __launch_bounds__(256) qk_row_norm_append_kernel(ST* __restrict__ proj, long long stride, const float* __restrict__ bias,
+                                                                 const float* __restrict__ q_gain, const float* __restrict__ k_gain, float temp_coef,
+                                                                 float temp_every, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
+                                                                 const int* __restrict__ block_table, int max_blocks, ST* __restrict__ kpool,
+                                                                 ST* __restrict__ vpool, float eps, int NQ, int NK, int NV, int page) {
+  __shared__ float red[33];
+  const int t = blockIdx.x, part = blockIdx.y, pos = tok_pos[t];
+  const int c0 = part == 0 ? 0 : part == 1 ? NQ : NQ + NK, n = part == 0 ? NQ : part == 1 ? NK : NV;
+  ST* src = proj + (size_t)t * stride + c0;
+  const float* b = bias != nullptr ? bias + c0 : nullptr;
+  ST* dst = src;
+  if (part != 0) {
+    const size_t cell = (size_t)block_table[(size_t)tok_slot[t] * max_blocks + pos / page] * page + (pos % page);
+    dst = (part == 1 ? kpool : vpool) + cell * n;
+  }
+  float r = 1.f;
+  const float* gain = part == 0 ? q_gain : part == 1 ? k_gain : nullptr;
+  if (part != 2) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+      float x[V];
+      load_biased<ST, V>(x, src, b, i);
+#pragma unroll
+      for (int v = 0; v < V; ++v) ss += x[v] * x[v];
+    }
+    r = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+    if (part == 0 && temp_coef != 0.f) r *= 1.f + temp_coef * logf(floorf((float)(pos + 1) / temp_every) + 1.f);
+  }
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {  // q: every thread overwrites only what it reads itself
+    float x[V];
+    load_biased<ST, V>(x, src, b, i);
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[v] *= gain != nullptr ? r * gain[i + v] : r;
+    if constexpr (V == 4) st4(dst + i, make_float4(x[0], x[1], x[2], x[3]));
+    else stf(dst + i, x[0]);
+  }
+}
+
+// out[t, i] = max(in[t, i] + bias[i], 0)^2 (bias may be null); V adjacent columns per thread
+template <typename ST, int V>
+__global__ void bias_relu_squared_kernel(ST* __restrict__ out, long long out_stride, const ST* __restrict__ in, long long in_stride,
+                                         const float* __restrict__ bias, int ff) {
+  const int t = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (i >= ff) return;
+  const ST* p = in + (size_t)t * in_stride;
+  ST* o = out + (size_t)t * out_stride + i;
+#pragma unroll
+  for (int k = 0; k < V; k += 4) {
+    float x[V < 4 ? V : 4];
+    load_biased<ST, (V < 4 ? V : 4)>(x, p, bias, i + k);
+#pragma unroll
+    for (int v = 0; v < (V < 4 ? V : 4); ++v) {
+      x[v] = fmaxf(x[v], 0.f);
+      x[v] *= x[v];
+    }
+    if constexpr (V >= 4) st4(o + k, make_float4(x[0], x[1], x[2], x[3]));
+    else stf(o, x[0]);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------------
 // Router of a mixture of experts: fp32 logits z = W_r h, scores = softmax(z) over all experts, the `top` largest scores are kept (ties: the
 // lower index) as they are (no renormalisation).  One block per token; a warp per expert for the dot products.
 //   route [tokens][E] fp32: the score of a chosen expert, 0 elsewhere;   top_idx / top_w [tokens][top]: the chosen experts, best first
@@ -309,9 +390,9 @@ constexpr int kRouterEPW = 4;
 // Grouped sigmoid routing of one token by one warp.  zk [3 E]: logits in, then choice scores | scores | group scores.
 //   s_e = sigmoid(z_e); choice c_e = s_e + correction_e; experts form `groups` equal runs of neighbours, a group's score is the sum of its two
 //   largest choice scores (its only one, for groups of one); only experts of the `keep` best groups can be chosen (ties: the lower index);
-//   the `top` largest choices win, weighted with s_e / (sum of the winners' s + 1e-20).
+//   the `top` largest choices win, weighted with w_scale s_e / (sum of the winners' s + 1e-20), or (renorm = 0) w_scale s_e.
 __device__ __forceinline__ void route_sigmoid_groups(float* __restrict__ zk, float* __restrict__ route_t, int* __restrict__ idx_t, float* __restrict__ w_t,
-                                                     const float* __restrict__ correction, int E, int top, int groups, int keep, int lane) {
+                                                     const float* __restrict__ correction, int E, int top, int groups, int keep, int renorm, float w_scale, int lane) {
   float* sc = zk + E;
   float* gs = zk + 2 * E;
   const int per = E / groups;
@@ -372,7 +453,7 @@ __device__ __forceinline__ void route_sigmoid_groups(float* __restrict__ zk, flo
     }
     __syncwarp();
   }
-  const float inv = 1.f / (total + 1e-20f);
+  const float inv = renorm ? w_scale / (total + 1e-20f) : w_scale;
   if (lane == 0)
     for (int j = 0; j < top; ++j) {
       const float wv = sc[idx_t[j]] * inv;
@@ -384,7 +465,7 @@ __device__ __forceinline__ void route_sigmoid_groups(float* __restrict__ zk, flo
 template <typename ST, int TOK>
 __global__ void __launch_bounds__(256) moe_router_kernel(float* __restrict__ route, int* __restrict__ top_idx, float* __restrict__ top_w,
                                                          const ST* __restrict__ h, const float* __restrict__ w_router, int T, int W, int E, int top,
-                                                         int zs, int mode, const float* __restrict__ correction, int groups, int keep) {
+                                                         int zs, int mode, const float* __restrict__ correction, int groups, int keep, int renorm, float w_scale) {
   // TOK tokens per block (rows h [TOK][W] in shared memory, storage type) and kRouterEPW experts per warp: a router word read from global
   // memory meets TOK rows, a row word read from shared memory meets kRouterEPW experts.  The dot product of a (token, expert) pair is summed
   // in the same order (lane-strided partial sums, then a shuffle tree) whatever else the block holds.  Scores [TOK][E] follow the rows.
@@ -429,7 +510,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(float* __restrict__ rou
     const size_t t = t0 + k;
     float* zk = z + k * zs;
     if (mode == 1) {
-      route_sigmoid_groups(zk, route + t * E, top_idx + t * top, top_w + t * top, correction, E, top, groups, keep, lane);
+      route_sigmoid_groups(zk, route + t * E, top_idx + t * top, top_w + t * top, correction, E, top, groups, keep, renorm, w_scale, lane);
       continue;
     }
     float mx = -INFINITY;
@@ -456,9 +537,9 @@ __global__ void __launch_bounds__(256) moe_router_kernel(float* __restrict__ rou
         if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
       }
       if (lane == 0) {
-        route[t * E + bi] = best;
+        route[t * E + bi] = best * w_scale;
         top_idx[t * top + j] = bi;
-        top_w[t * top + j] = best;
+        top_w[t * top + j] = best * w_scale;
         zk[bi] = -1.f;  // scores are positive: taken
       }
       __syncwarp();
@@ -1068,8 +1149,43 @@ int qs_hyb_qk_prepare_append(void* proj, int64_t stride, const float* bias, cons
   return check_cuda(cudaGetLastError(), "hyb_qk_prepare_append");
 }
 
+int qs_hyb_qk_row_norm_append(void* proj, int64_t stride, const float* bias, const float* q_gain, const float* k_gain, float temp_coef, float temp_every,
+                              const int32_t* tok_slot, const int32_t* tok_pos, const int32_t* block_table, int max_blocks, void* kpool, void* vpool,
+                              float eps, int tokens_n, int q_cols, int k_cols, int v_cols, int page_size, int dtype, void* stream) {
+  QS_REQUIRE(proj && q_gain && k_gain && tok_slot && tok_pos && block_table && kpool && vpool, "hyb_qk_row_norm_append: null tensor");
+  QS_REQUIRE(q_cols > 0 && k_cols > 0 && v_cols > 0 && page_size > 0 && (temp_coef == 0.f || temp_every > 0.f), "hyb_qk_row_norm_append: bad sizes");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool v4 = q_cols % 4 == 0 && k_cols % 4 == 0 && v_cols % 4 == 0 && stride % 4 == 0 && al16(proj) && al16(kpool) && al16(vpool);
+  dim3 grid(tokens_n, 3);
+#define QS_LAUNCH(ST, V)                                                                                                                         \
+  qk_row_norm_append_kernel<ST, V><<<grid, 256, 0, s>>>((ST*)proj, stride, bias, q_gain, k_gain, temp_coef, temp_every, tok_slot, tok_pos,        \
+                                                        block_table, max_blocks, (ST*)kpool, (ST*)vpool, eps, q_cols, k_cols, v_cols, page_size)
+  if (v4) QS_DT(dtype, (QS_LAUNCH(__nv_bfloat16, 4)), (QS_LAUNCH(float, 4)));
+  else QS_DT(dtype, (QS_LAUNCH(__nv_bfloat16, 1)), (QS_LAUNCH(float, 1)));
+#undef QS_LAUNCH
+  return check_cuda(cudaGetLastError(), "hyb_qk_row_norm_append");
+}
+
+int qs_hyb_bias_relu_squared(void* out, int64_t out_stride, const void* in, int64_t in_stride, const float* bias, int tokens_n, int ff, int dtype,
+                             void* stream) {
+  QS_REQUIRE(out && in && ff > 0, "hyb_bias_relu_squared: null tensor");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool v8 = ff % 8 == 0 && out_stride % 8 == 0 && in_stride % 8 == 0 && al16(out) && al16(in);
+  const int per = v8 ? 8 : 1;
+  dim3 grid(tokens_n, (ff / per + 255) / 256);
+#define QS_LAUNCH(ST, V) bias_relu_squared_kernel<ST, V><<<grid, 256, 0, s>>>((ST*)out, out_stride, (const ST*)in, in_stride, bias, ff)
+  if (v8) QS_DT(dtype, (QS_LAUNCH(__nv_bfloat16, 8)), (QS_LAUNCH(float, 8)));
+  else QS_DT(dtype, (QS_LAUNCH(__nv_bfloat16, 1)), (QS_LAUNCH(float, 1)));
+#undef QS_LAUNCH
+  return check_cuda(cudaGetLastError(), "hyb_bias_relu_squared");
+}
+
 int qs_hyb_moe_router(float* route, int32_t* top_idx, float* top_w, const void* h, const float* w_router, int tokens_n, int width, int experts,
-                      int top, int mode, const float* correction, int groups, int keep, int dtype, void* stream) {
+                      int top, int mode, const float* correction, int groups, int keep, int renorm, float w_scale, int dtype, void* stream) {
   QS_REQUIRE(route && top_idx && top_w && h && w_router, "hyb_moe_router: null tensor");
   QS_REQUIRE(experts >= 1 && top >= 1 && top <= experts, "hyb_moe_router: 1 <= top <= experts");
   QS_REQUIRE(mode == QS_ROUTER_SOFTMAX || mode == QS_ROUTER_SIGMOID_GROUPS, "hyb_moe_router: unknown mode");
@@ -1090,7 +1206,7 @@ int qs_hyb_moe_router(float* route, int32_t* top_idx, float* top_w, const void* 
   do {                                                                                                                                  \
     if (smb > 48 * 1024) cudaFuncSetAttribute(moe_router_kernel<ST, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smb);       \
     moe_router_kernel<ST, TOK><<<(tokens_n + TOK - 1) / TOK, 256, smb, s>>>(route, top_idx, top_w, (const ST*)h, w_router, tokens_n,   \
-                                                                          width, experts, top, zs, mode, correction, groups, keep);    \
+                                                                          width, experts, top, zs, mode, correction, groups, keep, renorm, w_scale);    \
   } while (0)
 #define QS_LAUNCH_T(ST)                          \
   switch (tok) {                                 \

@@ -47,6 +47,9 @@ __device__ __forceinline__ float block_max(float v, float* red) {
   return warp_max(t);
 }
 
+// floats of a prepared row of the state-space layer: [H*Dv x | G*N B | G*N C | H dt | H decay], padded to whole 16-byte words
+__host__ __device__ __forceinline__ int ssd_row_floats(int H, int G, int N, int Dv) { return (H * Dv + 2 * G * N + 2 * H + 3) & ~3; }
+
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
 // four elements of the storage type at once
@@ -157,4 +160,9 @@ __device__ __forceinline__ void cap_scores(float (&s)[N][4], float in, float out
 }
 
 }  // namespace hyb
+
+// hybrid_linear.cu: S <- a S + B (dt x)^T, o = S^T C + skip_h x over prepared rows (ssd_row_floats); state fp32 [slots][H][N][Dv]
+int ssd_scan(float* o_raw, const float* prep, float* state, const float* skip, const int* entry_start, const int* entry_len, const int* entry_slot,
+             const int* entry_pos0, int T, int E, int H, int G, int N, int Dv, cudaStream_t s);
+
 }  // namespace qs

@@ -3,8 +3,10 @@
 //   gate recurrence (HGRN2):  S <- diag(f) S + (1 - f) v^T,  o = S^T q      f per (head, row): the forget gate also sets the write strength
 //   retention:                S <- decay_h S + k v^T,        o = S^T q      one fixed decay per head, rotary q / k
 //   gated linear attention:   S <- diag(a) S + k v^T,        o = S^T q      a per (head, row) from a low-rank projection of the input
+//   state space:              S <- a S + B (dt x)^T,         y = S^T C + D x   a and dt per (token, head), B and C shared by groups of heads
+//                             (its first and last step are in hybrid_recurrent.cu)
 //
-// Both run in three steps on the flat token batch (hybrid.cu describes the batch tables):
+// All run in three steps on the flat token batch (hybrid.cu describes the batch tables):
 //   1. prepare: projection rows -> fp32 rows [H*D q | H*D g | H*Dv v]  (g = f, or the rotated and scaled k; gated linear attention has
 //      three row vectors: [H*D q | H*D k | H*D a | H*Dv v]); everything that enters the recurrence is fp32 from here on
 //   2. scan: one block per (entry, head, block of state columns) walks the entry's tokens in order with its columns of S in registers; a run
@@ -105,7 +107,9 @@ __global__ void gated_linear_prepare_kernel(float* __restrict__ prep, const ST* 
 //   MODE kScanHeadDecay:    S_i <- decay S_i + g_i v
 //   MODE kScanChannelGate:  S_i <- g_i S_i + (1 - g_i) v   (written as v + g_i (S_i - v))
 //   MODE kScanChannelDecay: S_i <- a_i S_i + g_i v         (a third row vector a follows g in the prepared row)
-//   o = sum_i S_i q_i
+//   MODE kScanTokenDecay:   S_i <- a S_i + g_i (dt v)      (dt and a: two numbers per (token, head) behind the prepared row's vectors; q and g are
+//                           shared by runs of H / G heads; prepared row [H*Dv v | G*D g | G*D q | H dt | H a], padded to a multiple of 4)
+//   o = sum_i S_i q_i      (kScanTokenDecay: + skip_h v)
 // ---------------------------------------------------------------------------------------------------------------------------------
 template <int PARTS>
 __device__ __forceinline__ float part_sum(float v) {
@@ -114,23 +118,36 @@ __device__ __forceinline__ float part_sum(float v) {
   return v;
 }
 
-constexpr int kScanHeadDecay = 0, kScanChannelGate = 1, kScanChannelDecay = 2;
+constexpr int kScanHeadDecay = 0, kScanChannelGate = 1, kScanChannelDecay = 2, kScanTokenDecay = 3;
+
+// floats of a prepared row; G: heads that have a q / g of their own
+__host__ __device__ __forceinline__ int scan_row_floats(int mode, int H, int G, int D, int Dv) {
+  if (mode == kScanTokenDecay) return ssd_row_floats(H, G, D, Dv);
+  return (mode == kScanChannelDecay ? 3 : 2) * H * D + H * Dv;
+}
 
 template <int DP, int PARTS, int CH, int CPT, int MODE, bool VEC>  // VEC: 16-byte staging (D, Dv, the prepared row and its base allow it)
 __global__ void __launch_bounds__(128) linear_scan_kernel(float* __restrict__ o_raw, const float* __restrict__ prep, float* __restrict__ state,
                                                           const float* __restrict__ head_decay, const int* __restrict__ entry_start,
                                                           const int* __restrict__ entry_len, const int* __restrict__ entry_slot,
-                                                          const int* __restrict__ entry_pos0, int H, int D, int Dv) {
+                                                          const int* __restrict__ entry_pos0, int H, int G, int D, int Dv) {
+  // head_decay [H]: kScanHeadDecay the decay, kScanTokenDecay the skip factor
   extern __shared__ __align__(16) float sm[];  // [2][CH][ROW]
+  constexpr bool TOKEN = MODE == kScanTokenDecay;
   constexpr int Q = DP / PARTS, SEG = Q + 4, COLS = 128 / PARTS * CPT;  // a part's q / g segment is padded by 16 bytes: parts hit different banks
   constexpr int NVEC = MODE == kScanChannelDecay ? 3 : 2;  // row vectors of a token: q, g [, a]
-  constexpr int QK = PARTS * SEG, ROW = NVEC * QK + COLS;
+  constexpr int QK = PARTS * SEG, ROW = NVEC * QK + COLS + (TOKEN ? 4 : 0);
   const int e = blockIdx.x, h = blockIdx.y, cg = blockIdx.z;
   const int tid = threadIdx.x, part = tid % PARTS, cl = tid / PARTS, col0 = cg * COLS + cl * CPT;  // CPT adjacent columns per thread
-  const int HD = H * D, P = NVEC * HD + H * Dv;
+  const int GD = G * D, P = scan_row_floats(MODE, H, G, D, Dv);
+  const int gh = TOKEN ? h / (H / G) : h;
+  // where vector `which` of the head, its values and its numbers dt, a lie in a prepared row
+  auto vec_at = [&](int which) { return TOKEN ? H * Dv + (1 - which) * GD + gh * D : which * GD + h * D; };
+  const int val_at = (TOKEN ? 0 : NVEC * GD) + h * Dv, num_at = H * Dv + 2 * GD + h;
   const int n = entry_len[e], s0 = entry_start[e];
   const bool fresh = entry_pos0[e] == 0;
-  const float decay = MODE == kScanHeadDecay ? head_decay[h] : 0.f;
+  float decay = MODE == kScanHeadDecay ? head_decay[h] : 0.f;
+  const float skip = TOKEN ? head_decay[h] : 0.f;
   float* Sg = state + ((size_t)entry_slot[e] * H + h) * (size_t)D * Dv;
   float S[CPT][Q];
 #pragma unroll
@@ -141,42 +158,48 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(float* __restrict__ o_
       S[c][j] = (col0 + c < Dv && !fresh && i < D) ? Sg[(size_t)i * Dv + col0 + c] : 0.f;
     }
   auto stage = [&](int chunk, int buf) {
+    const int cnt = min(CH, n - chunk * CH);  // tokens of the chunk (the rest of the buffer is not read)
     if (VEC) {
-      constexpr int QV = Q / 4, NQK = NVEC * PARTS * QV, NV = COLS / 4, ITEMS = NQK + NV;
-      for (int idx = tid; idx < CH * ITEMS; idx += 128) {
+      constexpr int QV = Q / 4, NQK = NVEC * PARTS * QV, NV = COLS / 4, ITEMS = NQK + NV + (TOKEN ? 2 : 0);
+      for (int idx = tid; idx < cnt * ITEMS; idx += 128) {
         const int tk = idx / ITEMS, j = idx - tk * ITEMS, t = chunk * CH + tk;
         float* base = sm + (size_t)(buf * CH + tk) * ROW;
-        const float* row = prep + (size_t)(s0 + min(t, n - 1)) * P;
+        const float* row = prep + (size_t)(s0 + t) * P;
         float* dst;
         const float* src = nullptr;
+        if (TOKEN && j >= NQK + NV) {  // dt, a
+          const int w = j - NQK - NV;
+          cp_async4(base + NVEC * QK + COLS + w, row + num_at + w * H);
+          continue;
+        }
         if (j < NQK) {
           const int which = j / (PARTS * QV), rem = j - which * (PARTS * QV), pp = rem / QV, w4 = rem - pp * QV, i = pp * Q + w4 * 4;
           dst = base + which * QK + pp * SEG + w4 * 4;
-          if (i < D) src = row + (size_t)which * HD + (size_t)h * D + i;
+          if (i < D) src = row + vec_at(which) + i;
         } else {
           const int c4 = (j - NQK) * 4, c = cg * COLS + c4;
           dst = base + NVEC * QK + c4;
-          if (c < Dv) src = row + NVEC * HD + (size_t)h * Dv + c;
+          if (c < Dv) src = row + val_at + c;
         }
-        if (t < n && src != nullptr) cp_async16(dst, src);
+        if (src != nullptr) cp_async16(dst, src);
         else *reinterpret_cast<float4*>(dst) = make_float4(0.f, 0.f, 0.f, 0.f);
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
       return;
     }
-    for (int idx = tid; idx < CH * ROW; idx += 128) {
+    for (int idx = tid; idx < cnt * ROW; idx += 128) {
       const int tk = idx / ROW, j = idx - tk * ROW, t = chunk * CH + tk;
       float* dst = sm + (size_t)(buf * CH + tk) * ROW + j;
       const float* src = nullptr;
-      if (t < n) {
-        const float* row = prep + (size_t)(s0 + t) * P;
-        if (j < NVEC * QK) {
-          const int which = j / QK, jj = j - which * QK, pp = jj / SEG, w = jj - pp * SEG, i = pp * Q + w;  // q (which = 0), g or a row i
-          if (w < Q && i < D) src = row + (size_t)which * HD + (size_t)h * D + i;
-        } else {
-          const int c = cg * COLS + j - NVEC * QK;
-          if (c < Dv) src = row + NVEC * HD + (size_t)h * Dv + c;
-        }
+      const float* row = prep + (size_t)(s0 + t) * P;
+      if (j < NVEC * QK) {
+        const int which = j / QK, jj = j - which * QK, pp = jj / SEG, w = jj - pp * SEG, i = pp * Q + w;  // q (which = 0), g or a row i
+        if (w < Q && i < D) src = row + vec_at(which) + i;
+      } else if (j < NVEC * QK + COLS) {
+        const int c = cg * COLS + j - NVEC * QK;
+        if (c < Dv) src = row + val_at + c;
+      } else if (j < NVEC * QK + COLS + 2) {
+        src = row + num_at + (j - NVEC * QK - COLS) * H;
       }
       if (src != nullptr) cp_async4(dst, src);
       else *dst = 0.f;
@@ -199,10 +222,16 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(float* __restrict__ o_
       const float4* q4 = reinterpret_cast<const float4*>(r + part * SEG);
       const float4* g4 = reinterpret_cast<const float4*>(r + QK + part * SEG);
       const float4* a4 = reinterpret_cast<const float4*>(r + (NVEC - 1) * QK + part * SEG);  // read in kScanChannelDecay only
-      float v[CPT], op[CPT][4];
+      float v[CPT], op[CPT][4], pass[CPT];
+      const float dt = TOKEN ? r[NVEC * QK + COLS] : 1.f;
+      if (TOKEN) decay = r[NVEC * QK + COLS + 1];
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
         v[c] = r[NVEC * QK + cl * CPT + c];
+        if (TOKEN) {
+          pass[c] = skip * v[c];
+          v[c] *= dt;
+        }
         op[c][0] = op[c][1] = op[c][2] = op[c][3] = 0.f;
       }
       // a q / g word read from shared memory serves the thread's CPT columns
@@ -230,7 +259,8 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(float* __restrict__ o_
       }
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
-        const float o = part_sum<PARTS>((op[c][0] + op[c][1]) + (op[c][2] + op[c][3]));
+        float o = part_sum<PARTS>((op[c][0] + op[c][1]) + (op[c][2] + op[c][3]));
+        if (TOKEN) o += pass[c];
         if (part == 0 && col0 + c < Dv) o_raw[(size_t)(s0 + ch * CH + tk) * H * Dv + (size_t)h * Dv + col0 + c] = o;
       }
     }
@@ -269,18 +299,18 @@ __global__ void linear_out_kernel(ST* __restrict__ out, long long out_stride, co
 
 template <int MODE>
 int launch_scan(float* o_raw, const float* prep, float* state, const float* head_decay, const int* entry_start, const int* entry_len,
-                const int* entry_slot, const int* entry_pos0, int T, int E, int H, int D, int Dv, cudaStream_t s) {
+                const int* entry_slot, const int* entry_pos0, int T, int E, int H, int G, int D, int Dv, cudaStream_t s) {
   constexpr int NVEC = MODE == kScanChannelDecay ? 3 : 2;
-  const int P = NVEC * H * D + H * Dv;
+  const int P = scan_row_floats(MODE, H, G, D, Dv);
   const bool vec = D % 4 == 0 && Dv % 4 == 0 && P % 4 == 0 && (reinterpret_cast<uintptr_t>(prep) & 15) == 0;
 #define QS_SCAN(DP, PARTS, CH, CPT)                                                                                                           \
   do {                                                                                                                                        \
     constexpr int cols = 128 / PARTS * CPT;                                                                                                   \
-    const size_t smb = (size_t)2 * CH * (NVEC * PARTS * (DP / PARTS + 4) + cols) * sizeof(float);                                                \
+    const size_t smb = (size_t)2 * CH * (NVEC * PARTS * (DP / PARTS + 4) + cols + (MODE == kScanTokenDecay ? 4 : 0)) * sizeof(float);            \
     dim3 grid(E, H, (Dv + cols - 1) / cols);                                                                                                  \
     auto kern = vec ? linear_scan_kernel<DP, PARTS, CH, CPT, MODE, true> : linear_scan_kernel<DP, PARTS, CH, CPT, MODE, false>;                 \
     if (smb > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smb);                                   \
-    kern<<<grid, 128, smb, s>>>(o_raw, prep, state, head_decay, entry_start, entry_len, entry_slot, entry_pos0, H, D, Dv);                    \
+    kern<<<grid, 128, smb, s>>>(o_raw, prep, state, head_decay, entry_start, entry_len, entry_slot, entry_pos0, H, G, D, Dv);                 \
   } while (0)
   // rows of a column per thread: all of them up to 32, 32 or 16 above (the parts of a column meet through shuffles).  Long runs of tokens
   // (prompt portions) take two adjacent columns per thread where the head has the columns for it: a q / g word read from shared memory then
@@ -301,6 +331,12 @@ int launch_scan(float* o_raw, const float* prep, float* state, const float* head
 }
 
 }  // namespace
+
+int ssd_scan(float* o_raw, const float* prep, float* state, const float* skip, const int* entry_start, const int* entry_len, const int* entry_slot,
+             const int* entry_pos0, int T, int E, int H, int G, int N, int Dv, cudaStream_t s) {
+  return launch_scan<kScanTokenDecay>(o_raw, prep, state, skip, entry_start, entry_len, entry_slot, entry_pos0, T, E, H, G, N, Dv, s);
+}
+
 }  // namespace qs
 
 using namespace qs;
@@ -326,7 +362,7 @@ int qs_hyb_gate_recurrence(void* out, int64_t out_stride, float* prep, float* o_
   const int HD = heads * dim, HDv = heads * vdim;
   QS_DT(dtype, (gate_prepare_kernel<__nv_bfloat16><<<tokens_n, 256, 0, s>>>(prep, (const __nv_bfloat16*)proj, stride, f_bias, lower, HD, HDv)),
         (gate_prepare_kernel<float><<<tokens_n, 256, 0, s>>>(prep, (const float*)proj, stride, f_bias, lower, HD, HDv)));
-  if (int rc = launch_scan<kScanChannelGate>(o_raw, prep, state, nullptr, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, dim, vdim, s)) return rc;
+  if (int rc = launch_scan<kScanChannelGate>(o_raw, prep, state, nullptr, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, heads, dim, vdim, s)) return rc;
   const int warps = tokens_n * heads;
   QS_DT(dtype,
         (linear_out_kernel<__nv_bfloat16><<<(warps + 3) / 4, 128, 0, s>>>((__nv_bfloat16*)out, out_stride, o_raw, norm_w, nullptr, 0, tokens_n, heads,
@@ -350,7 +386,7 @@ int qs_hyb_retention(void* out, int64_t out_stride, float* prep, float* o_raw, c
                                                                            heads, dim, vdim)),
         (retention_prepare_kernel<float><<<tokens_n, 256, rot_dims * sizeof(float), s>>>(prep, (const float*)proj, stride, tok_pos, inv_freq, rot_dims, k_scale, heads, dim,
                                                                   vdim)));
-  if (int rc = launch_scan<kScanHeadDecay>(o_raw, prep, state, head_decay, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, dim, vdim, s)) return rc;
+  if (int rc = launch_scan<kScanHeadDecay>(o_raw, prep, state, head_decay, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, heads, dim, vdim, s)) return rc;
   const int warps = tokens_n * heads;
   const size_t gate_off = (size_t)2 * heads * dim + (size_t)heads * vdim;  // the output gate follows q | k | v in the projection row
   QS_DT(dtype,
@@ -375,7 +411,7 @@ int qs_hyb_gated_linear(void* out, int64_t out_stride, float* prep, float* o_raw
   QS_DT(dtype,
         (gated_linear_prepare_kernel<__nv_bfloat16><<<tokens_n, 256, 0, s>>>(prep, (const __nv_bfloat16*)proj, stride, z, z_bias, inv_tau, q_scale, HD, HDv)),
         (gated_linear_prepare_kernel<float><<<tokens_n, 256, 0, s>>>(prep, (const float*)proj, stride, z, z_bias, inv_tau, q_scale, HD, HDv)));
-  if (int rc = launch_scan<kScanChannelDecay>(o_raw, prep, state, nullptr, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, dim, vdim, s)) return rc;
+  if (int rc = launch_scan<kScanChannelDecay>(o_raw, prep, state, nullptr, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, heads, heads, dim, vdim, s)) return rc;
   const int warps = tokens_n * heads;
   const size_t gate_off = (size_t)2 * HD + (size_t)HDv;  // the output gate follows q | k | v in the projection row
   QS_DT(dtype,

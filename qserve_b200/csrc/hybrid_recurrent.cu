@@ -1,0 +1,463 @@
+// qserve_b200 -- recurrent layers of the hybrid decoders that read short causal convolutions.
+//
+//   state space (Mamba-2):  S <- a S + dt B x^T,  y = S^T C + D x    per head a [N, Dv] fp32 state; x, B, C pass a convolution and silu, a and dt are
+//                           one number per (token, head); y * silu(z) is brought to unit RMS in equal parts.  The scan itself is a mode of the
+//                           linear-scan kernel (hybrid_linear.cu); its first and last step are here.
+//   gated linear unit (RG-LRU):  S <- a S + sqrt(1 - a^2) i u        per channel one fp32 number; u is the convolved branch, a and i come from
+//                           block-diagonal projections of u (a batched product between the two kernels here); the output is S * gelu_tanh(y).
+//                           Runs of at least a tile of tokens are scanned tile by tile: every tile's own (product of a, end state from
+//                           zero) first, then the tiles' start states, then the tiles again from there.
+//
+// Batch tables: see hybrid.cu.  Convolution states (fp32): [slots][taps - 1][channels], oldest input first.
+#include <cuda_bf16.h>
+#include <math.h>
+
+#include <algorithm>
+
+#include "../../include/qserve_b200.h"
+#include "common.cuh"
+#include "hybrid_common.cuh"
+#include "launch.h"
+
+namespace qs {
+namespace {
+
+using namespace hyb;
+
+constexpr int kMaxTaps = 17;
+
+// The convolution's inputs of one token, channels c .. c + V - 1: `back` tokens before row t.  Inputs ahead of the portion come from the
+// convolution state, inputs ahead of the sequence are zero; `in_bias` (may be null) belongs to the inputs.
+template <typename ST, int V>
+__device__ __forceinline__ void conv_input(float (&x)[V], const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias,
+                                           const float* st, int t, int local, int pos, int back, int taps, int C, int c) {
+#pragma unroll
+  for (int v = 0; v < V; ++v) x[v] = 0.f;
+  if (pos - back < 0) return;
+  if (local - back >= 0) {
+    const ST* p = in + (size_t)(t - back) * stride + c;
+    if constexpr (V == 4) {
+      const float4 q = ld4(p);
+      x[0] = q.x; x[1] = q.y; x[2] = q.z; x[3] = q.w;
+    } else {
+      x[0] = ldf(p);
+    }
+    if (in_bias != nullptr) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) x[v] += in_bias[c + v];
+    }
+  } else {
+    const float* p = st + (size_t)(taps - 1 + local - back) * C + c;
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[v] = p[v];
+  }
+}
+
+// Convolution of row t at channels c .. c + V - 1 (bias included).  In a step of single tokens the thread is the only reader of its channels'
+// state and shifts the token's input in (`shift`); other steps do that in conv_state_kernel afterwards.
+template <typename ST, int V>
+__device__ __forceinline__ void conv_row(float (&y)[V], const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias, float* st,
+                                         const float* __restrict__ w, const float* __restrict__ b, int t, int local, int pos, int taps, int C, int c,
+                                         bool shift) {
+#pragma unroll
+  for (int v = 0; v < V; ++v) y[v] = b != nullptr ? b[c + v] : 0.f;
+  for (int j = 0; j < taps; ++j) {
+    float x[V];
+    conv_input<ST, V>(x, in, stride, in_bias, st, t, local, pos, taps - 1 - j, taps, C, c);
+#pragma unroll
+    for (int v = 0; v < V; ++v) y[v] += w[(size_t)(c + v) * taps + j] * x[v];
+    if (shift && j > 0) {  // input j is slot j - 1 of the next token's state; slot j is read before slot j is written
+#pragma unroll
+      for (int v = 0; v < V; ++v) st[(size_t)(j - 1) * C + c + v] = x[v];
+    }
+  }
+}
+
+// the sequence's convolution state after a portion: its last taps - 1 inputs (older ones shift out)
+template <typename ST>
+__global__ void conv_state_kernel(float* __restrict__ conv_state, const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias,
+                                  const int* __restrict__ entry_start, const int* __restrict__ entry_len, const int* __restrict__ entry_slot,
+                                  const int* __restrict__ entry_pos0, int C, int taps) {
+  const int e = blockIdx.y;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int n = entry_len[e], s0 = entry_start[e], keep = taps - 1;
+  float* st = conv_state + (size_t)entry_slot[e] * keep * C + c;
+  const bool fresh = entry_pos0[e] == 0;
+  const float bias = in_bias != nullptr ? in_bias[c] : 0.f;
+  for (int i = 0; i < keep; ++i) {  // slot i takes an input that lies further on in the old state: no slot is read after it was written
+    const int src = n - keep + i;   // index in the portion, negative: older than the portion
+    float v;
+    if (src >= 0) v = ldf(in + (size_t)(s0 + src) * stride + c) + bias;
+    else v = fresh ? 0.f : st[(size_t)(keep + src) * C];
+    st[(size_t)i * C] = v;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------------
+// state space, step 1.  projection row: [inner z | inner x | G*N B | G*N C | H dt], inner = H * Dv
+//   prepared row (ssd_row_floats): [inner x | G*N B | G*N C | H dt | H a]:  x, B, C convolved and through silu, dt <- softplus(dt + dt_bias),
+//   a = exp(-exp(A_log) dt)
+// grid (runs of `run` tokens, blocks of 128 V channels)
+// ---------------------------------------------------------------------------------------------------------------------------------
+template <typename ST, int V>
+__global__ void __launch_bounds__(128) ssd_prepare_kernel(float* __restrict__ prep, const ST* __restrict__ proj, long long stride,
+                                                          const float* __restrict__ conv_w, const float* __restrict__ conv_b, float* conv_state,
+                                                          const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                          const int* __restrict__ tok_entry, const int* __restrict__ tok_pos,
+                                                          const int* __restrict__ entry_start, const int* __restrict__ entry_slot, int T, int H, int G,
+                                                          int N, int Dv, int taps, int run, int shift) {
+  const int inner = H * Dv, C = inner + 2 * G * N, P = ssd_row_floats(H, G, N, Dv);
+  const int c = (blockIdx.y * 128 + threadIdx.x) * V;
+  const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+  for (int t = t0; t < t1; ++t) {
+    const int e = tok_entry[t];
+    float* o = prep + (size_t)t * P;
+    if (c < C) {
+      float y[V];
+      conv_row<ST, V>(y, proj + inner, stride, nullptr, conv_state + (size_t)entry_slot[e] * (taps - 1) * C, conv_w, conv_b, t, t - entry_start[e],
+                      tok_pos[t], taps, C, c, shift != 0);
+#pragma unroll
+      for (int v = 0; v < V; ++v) y[v] = silu_f(y[v]);
+      if constexpr (V == 4) st4(o + c, make_float4(y[0], y[1], y[2], y[3]));
+      else o[c] = y[0];
+    }
+    if (blockIdx.y == 0)
+      for (int h = threadIdx.x; h < H; h += 128) {
+        const float z = ldf(proj + (size_t)t * stride + inner + C + h) + dt_bias[h];
+        const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+        o[C + h] = dt;
+        o[C + H + h] = expf(-expf(a_log[h]) * dt);
+      }
+  }
+}
+
+// state space, step 3: y <- y * silu(z), unit RMS in equal parts of the row, times norm_w and a constant.  One block per (token, part); the part
+// waits in shared memory between its two passes.
+template <typename ST>
+__global__ void __launch_bounds__(256) ssd_out_kernel(ST* __restrict__ out, long long out_stride, const float* __restrict__ y, const ST* __restrict__ z,
+                                                      long long z_stride, const float* __restrict__ norm_w, float out_scale, float eps, int inner,
+                                                      int part, int vec) {
+  extern __shared__ __align__(16) float ys[];  // [part]
+  __shared__ float red[33];
+  const int t = blockIdx.x, c0 = blockIdx.y * part;
+  const float* yr = y + (size_t)t * inner + c0;
+  const ST* zr = z + (size_t)t * z_stride + c0;
+  ST* o = out + (size_t)t * out_stride + c0;
+  float ss = 0.f;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < part; i += blockDim.x * 4) {
+      float4 a = ld4(yr + i);
+      const float4 g = ld4(zr + i);
+      a.x *= silu_f(g.x); a.y *= silu_f(g.y); a.z *= silu_f(g.z); a.w *= silu_f(g.w);
+      ss += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
+      st4(ys + i, a);
+    }
+  } else {
+    for (int i = threadIdx.x; i < part; i += blockDim.x) {
+      const float a = yr[i] * silu_f(ldf(zr + i));
+      ss += a * a;
+      ys[i] = a;
+    }
+  }
+  const float r = out_scale / sqrtf(block_sum(ss, red) / (float)part + eps);
+  if (vec) {  // every thread reads back what it wrote itself
+    for (int i = threadIdx.x * 4; i < part; i += blockDim.x * 4) {
+      const float4 a = ld4(ys + i), w = ld4(norm_w + c0 + i);
+      st4(o + i, make_float4(a.x * r * w.x, a.y * r * w.y, a.z * r * w.z, a.w * r * w.w));
+    }
+  } else {
+    for (int i = threadIdx.x; i < part; i += blockDim.x) stf(o + i, ys[i] * r * norm_w[c0 + i]);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------------
+// gated linear unit.  projection row: [W y | W x] (biases not yet added)
+// step 1: u = convolution of x + x_bias, in the storage type [T][W]
+// ---------------------------------------------------------------------------------------------------------------------------------
+template <typename ST, int V>
+__global__ void __launch_bounds__(128) lru_conv_kernel(ST* __restrict__ u, const ST* __restrict__ proj, long long stride, const float* __restrict__ x_bias,
+                                                       const float* __restrict__ conv_w, const float* __restrict__ conv_b, float* conv_state,
+                                                       const int* __restrict__ tok_entry, const int* __restrict__ tok_pos,
+                                                       const int* __restrict__ entry_start, const int* __restrict__ entry_slot, int T, int W, int taps,
+                                                       int run, int shift) {
+  const int c = (blockIdx.y * 128 + threadIdx.x) * V;
+  if (c >= W) return;
+  const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+  for (int t = t0; t < t1; ++t) {
+    const int e = tok_entry[t];
+    float y[V];
+    conv_row<ST, V>(y, proj + W, stride, x_bias, conv_state + (size_t)entry_slot[e] * (taps - 1) * W, conv_w, conv_b, t, t - entry_start[e], tok_pos[t],
+                    taps, W, c, shift != 0);
+    if constexpr (V == 4) st4(u + (size_t)t * W + c, make_float4(y[0], y[1], y[2], y[3]));
+    else stf(u + (size_t)t * W + c, y[0]);
+  }
+}
+
+// step 2 (between the kernels): gate logits z fp32 [blocks][T][2 W / blocks]: a block's r logits, then its i logits.
+// step 3: the recurrence.  One token of one channel: r = sigmoid(z_r + r_bias), i = sigmoid(z_i + i_bias), log a = rate * r (rate < 0 per
+// channel), S <- a S + sqrt(1 - a^2) i u with 1 - a^2 = -expm1(2 log a).
+struct LruChannel {
+  const float* zr;    // r logit of row 0; rows are zs floats apart
+  size_t zs, zi;      // zi: distance of the i logit
+  float rb, ib, rate;
+};
+__device__ __forceinline__ LruChannel lru_channel(const float* z, const float* r_bias, const float* i_bias, const float* rate, int T, int W, int blocks,
+                                                  int c) {
+  const int wb = W / blocks, b = c / wb, j = c - b * wb;
+  LruChannel k;
+  k.zr = z + (size_t)b * T * 2 * wb + j;
+  k.zs = 2 * (size_t)wb;
+  k.zi = wb;
+  k.rb = r_bias[c];
+  k.ib = i_bias[c];
+  k.rate = rate[c];
+  return k;
+}
+__device__ __forceinline__ void lru_gates(float& a, float& b, float zr, float zi, float u, const LruChannel& k) {
+  const float la = k.rate * sigmoid_f(zr + k.rb);
+  a = expf(la);
+  b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + k.ib) * u;
+}
+
+constexpr int kLruBatch = 4;  // tokens whose inputs are on their way at once
+
+// what a tile of rows does to a state: S <- A S + B.  sums [n_tiles][2][W]
+template <typename ST>
+__global__ void __launch_bounds__(128) lru_tile_sums_kernel(float* __restrict__ sums, const ST* __restrict__ u, const float* __restrict__ z,
+                                                            const float* __restrict__ r_bias, const float* __restrict__ i_bias,
+                                                            const float* __restrict__ rate, const int* __restrict__ tile_entry,
+                                                            const int* __restrict__ tile_row0, const int* __restrict__ entry_start,
+                                                            const int* __restrict__ entry_len, int T, int W, int blocks, int tile_rows) {
+  const int c = blockIdx.y * 128 + threadIdx.x, tile = blockIdx.x;
+  if (c >= W) return;
+  const int e = tile_entry[tile], r0 = tile_row0[tile], n = min(tile_rows, entry_len[e] - r0), s0 = entry_start[e] + r0;
+  const LruChannel k = lru_channel(z, r_bias, i_bias, rate, T, W, blocks, c);
+  float A = 1.f, S = 0.f;
+  for (int j = 0; j < n; j += kLruBatch) {
+    float zr[kLruBatch], zi[kLruBatch], uu[kLruBatch];
+#pragma unroll
+    for (int q = 0; q < kLruBatch; ++q) {
+      const size_t t = s0 + min(j + q, n - 1);
+      zr[q] = k.zr[t * k.zs];
+      zi[q] = k.zr[t * k.zs + k.zi];
+      uu[q] = ldf(u + t * W + c);
+    }
+#pragma unroll
+    for (int q = 0; q < kLruBatch; ++q) {
+      if (j + q >= n) break;
+      float a, b;
+      lru_gates(a, b, zr[q], zi[q], uu[q], k);
+      A *= a;
+      S = a * S + b;
+    }
+  }
+  sums[(size_t)tile * 2 * W + c] = A;
+  sums[((size_t)tile * 2 + 1) * W + c] = S;
+}
+
+// start state of every tile, over the tile's A.  An entry's tiles are neighbours; the block of its first tile walks them.
+__global__ void __launch_bounds__(128) lru_tile_starts_kernel(float* __restrict__ sums, const float* __restrict__ state, const int* __restrict__ tile_entry,
+                                                              const int* __restrict__ tile_row0, const int* __restrict__ entry_slot,
+                                                              const int* __restrict__ entry_pos0, int n_tiles, int W) {
+  const int c = blockIdx.y * 128 + threadIdx.x;
+  int tile = blockIdx.x;
+  if (tile_row0[tile] != 0 || c >= W) return;
+  const int e = tile_entry[tile];
+  float S = entry_pos0[e] == 0 ? 0.f : state[(size_t)entry_slot[e] * W + c];
+  do {
+    float* p = sums + (size_t)tile * 2 * W + c;
+    const float A = p[0], B = p[W];
+    p[0] = S;
+    S = A * S + B;
+    ++tile;
+  } while (tile < n_tiles && tile_entry[tile] == e);
+}
+
+// The recurrence over a tile (tiles != 0: start state from sums) or over a whole entry of fewer than long_min tokens (tiles == 0: start state
+// from the slot; longer entries are left to the tiles), read out through the gelu branch.  The slot takes the state after the entry's last row.
+template <typename ST>
+__global__ void __launch_bounds__(128) lru_scan_kernel(ST* __restrict__ out, long long out_stride, float* state, const float* __restrict__ sums,
+                                                       const ST* __restrict__ u, const float* __restrict__ z, const ST* __restrict__ y, long long y_stride,
+                                                       const float* __restrict__ y_bias, const float* __restrict__ r_bias,
+                                                       const float* __restrict__ i_bias, const float* __restrict__ rate,
+                                                       const int* __restrict__ tile_entry, const int* __restrict__ tile_row0,
+                                                       const int* __restrict__ entry_start, const int* __restrict__ entry_len,
+                                                       const int* __restrict__ entry_slot, const int* __restrict__ entry_pos0, int tiles, int long_min, int T,
+                                                       int W, int blocks, int tile_rows) {
+  const int c = blockIdx.y * 128 + threadIdx.x;
+  const int e = tiles ? tile_entry[blockIdx.x] : blockIdx.x;
+  const int len = entry_len[e], r0 = tiles ? tile_row0[blockIdx.x] : 0, n = tiles ? min(tile_rows, len - r0) : len;
+  if (c >= W || (!tiles && len >= long_min)) return;
+  const int s0 = entry_start[e] + r0;
+  float* slot = state + (size_t)entry_slot[e] * W + c;
+  const LruChannel k = lru_channel(z, r_bias, i_bias, rate, T, W, blocks, c);
+  const float yb = y_bias[c];
+  float S = tiles ? sums[(size_t)blockIdx.x * 2 * W + c] : (entry_pos0[e] == 0 ? 0.f : *slot);
+  for (int j = 0; j < n; j += kLruBatch) {
+    float zr[kLruBatch], zi[kLruBatch], uu[kLruBatch], yy[kLruBatch];
+#pragma unroll
+    for (int q = 0; q < kLruBatch; ++q) {
+      const size_t t = s0 + min(j + q, n - 1);
+      zr[q] = k.zr[t * k.zs];
+      zi[q] = k.zr[t * k.zs + k.zi];
+      uu[q] = ldf(u + t * W + c);
+      yy[q] = ldf(y + t * y_stride + c);
+    }
+#pragma unroll
+    for (int q = 0; q < kLruBatch; ++q) {
+      if (j + q >= n) break;
+      float a, b;
+      lru_gates(a, b, zr[q], zi[q], uu[q], k);
+      S = a * S + b;
+      const float g = yy[q] + yb;  // gelu_tanh(g) = g / (1 + e^(-2 sqrt(2/pi) (g + 0.044715 g^3)))
+      stf(out + (size_t)(s0 + j + q) * out_stride + c, S * (g / (1.f + expf(-2.f * 0.7978845608028654f * (g + 0.044715f * g * g * g)))));
+    }
+  }
+  if (r0 + n == len) *slot = S;
+}
+
+template <typename ST>
+int launch_conv_state(float* conv_state, const ST* in, long long stride, const float* in_bias, const int* entry_start, const int* entry_len,
+                      const int* entry_slot, const int* entry_pos0, int E, int C, int taps, cudaStream_t s) {
+  if (taps > 1)
+    conv_state_kernel<ST><<<dim3((C + 127) / 128, E), 128, 0, s>>>(conv_state, in, stride, in_bias, entry_start, entry_len, entry_slot, entry_pos0, C, taps);
+  return check_cuda(cudaGetLastError(), "hyb convolution state");
+}
+
+bool aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+
+// tokens a block of a convolution kernel walks: neighbours find each other's rows in the cache once there are blocks enough
+int conv_run(int T) { return T >= 2048 ? 8 : T >= 512 ? 4 : 1; }
+
+template <typename ST>
+int launch_state_space(void* out, long long out_stride, float* prep, float* o_raw, const void* proj_, long long stride, const float* conv_w,
+                       const float* conv_b, float* conv_state, float* state, const float* a_log, const float* dt_bias, const float* skip,
+                       const float* norm_w, int norm_groups, float out_scale, const int* tok_entry, const int* tok_pos, const int* entry_start,
+                       const int* entry_len, const int* entry_slot, const int* entry_pos0, int T, int E, int H, int G, int N, int Dv, int taps, float eps,
+                       cudaStream_t s) {
+  const ST* proj = static_cast<const ST*>(proj_);
+  const int inner = H * Dv, C = inner + 2 * G * N, run = conv_run(T), shift = T == E && taps > 1;
+  const bool v4 = C % 4 == 0 && inner % 4 == 0 && stride % 4 == 0 && aligned(proj, 4 * sizeof(ST)) && aligned(prep, 16);
+  dim3 grid((T + run - 1) / run, (C + (v4 ? 512 : 128) - 1) / (v4 ? 512 : 128));
+  auto prepare = v4 ? ssd_prepare_kernel<ST, 4> : ssd_prepare_kernel<ST, 1>;
+  prepare<<<grid, 128, 0, s>>>(prep, proj, stride, conv_w, conv_b, conv_state, a_log, dt_bias, tok_entry, tok_pos, entry_start, entry_slot, T, H, G, N, Dv,
+                               taps, run, shift);
+  if (!shift)
+    if (int rc = launch_conv_state<ST>(conv_state, proj + inner, stride, nullptr, entry_start, entry_len, entry_slot, entry_pos0, E, C, taps, s)) return rc;
+  if (int rc = ssd_scan(o_raw, prep, state, skip, entry_start, entry_len, entry_slot, entry_pos0, T, E, H, G, N, Dv, s)) return rc;
+  const int part = inner / norm_groups, threads = part >= 1024 ? 256 : 128;
+  const size_t smb = (size_t)part * sizeof(float);
+  const int vec = part % 4 == 0 && stride % 4 == 0 && out_stride % 4 == 0 && aligned(proj, 4 * sizeof(ST)) && aligned(out, 4 * sizeof(ST)) &&
+                  aligned(o_raw, 16) && aligned(norm_w, 16);
+  if (smb > 48 * 1024) cudaFuncSetAttribute(ssd_out_kernel<ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smb);
+  ssd_out_kernel<ST><<<dim3(T, norm_groups), threads, smb, s>>>((ST*)out, out_stride, o_raw, proj, stride, norm_w, out_scale, eps, inner, part, vec);
+  return check_cuda(cudaGetLastError(), "hyb_state_space");
+}
+
+template <typename ST>
+int launch_lru_conv(void* u, const void* proj_, long long stride, const float* x_bias, const float* conv_w, const float* conv_b, float* conv_state,
+                    const int* tok_entry, const int* tok_pos, const int* entry_start, const int* entry_len, const int* entry_slot, const int* entry_pos0,
+                    int T, int E, int W, int taps, cudaStream_t s) {
+  const ST* proj = static_cast<const ST*>(proj_);
+  const int run = conv_run(T), shift = T == E && taps > 1;
+  const bool v4 = W % 4 == 0 && stride % 4 == 0 && aligned(proj, 4 * sizeof(ST)) && aligned(u, 4 * sizeof(ST));
+  dim3 grid((T + run - 1) / run, (W + (v4 ? 512 : 128) - 1) / (v4 ? 512 : 128));
+  auto conv = v4 ? lru_conv_kernel<ST, 4> : lru_conv_kernel<ST, 1>;
+  conv<<<grid, 128, 0, s>>>((ST*)u, proj, stride, x_bias, conv_w, conv_b, conv_state, tok_entry, tok_pos, entry_start, entry_slot, T, W, taps, run, shift);
+  if (!shift) return launch_conv_state<ST>(conv_state, proj + W, stride, x_bias, entry_start, entry_len, entry_slot, entry_pos0, E, W, taps, s);
+  return check_cuda(cudaGetLastError(), "hyb_lru_conv");
+}
+
+template <typename ST>
+int launch_lru_scan(void* out, long long out_stride, float* state, float* sums, const void* u, const float* z, const void* proj, long long stride,
+                    const float* y_bias, const float* r_bias, const float* i_bias, const float* rate, const int* tile_entry, const int* tile_row0,
+                    int n_tiles, int n_short, const int* entry_start, const int* entry_len, const int* entry_slot, const int* entry_pos0, int T, int E,
+                    int W, int blocks, int tile_rows, int long_min, cudaStream_t s) {
+  const int cols = (W + 127) / 128;
+  if (n_tiles > 0) {
+    dim3 grid(n_tiles, cols);
+    lru_tile_sums_kernel<ST><<<grid, 128, 0, s>>>(sums, (const ST*)u, z, r_bias, i_bias, rate, tile_entry, tile_row0, entry_start, entry_len, T, W, blocks,
+                                                  tile_rows);
+    lru_tile_starts_kernel<<<grid, 128, 0, s>>>(sums, state, tile_entry, tile_row0, entry_slot, entry_pos0, n_tiles, W);
+    lru_scan_kernel<ST><<<grid, 128, 0, s>>>((ST*)out, out_stride, state, sums, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias, rate,
+                                             tile_entry, tile_row0, entry_start, entry_len, entry_slot, entry_pos0, 1, long_min, T, W, blocks, tile_rows);
+  }
+  if (n_short > 0)
+    lru_scan_kernel<ST><<<dim3(E, cols), 128, 0, s>>>((ST*)out, out_stride, state, nullptr, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias,
+                                                      rate, nullptr, nullptr, entry_start, entry_len, entry_slot, entry_pos0, 0, long_min, T, W, blocks,
+                                                      tile_rows);
+  return check_cuda(cudaGetLastError(), "hyb_lru_scan");
+}
+
+}  // namespace
+}  // namespace qs
+
+using namespace qs;
+
+#define QS_DT(dtype, CALL_BF16, CALL_F32)                                               \
+  do {                                                                                  \
+    if ((dtype) == QS_DTYPE_BF16) { CALL_BF16; }                                        \
+    else if ((dtype) == QS_DTYPE_F32) { CALL_F32; }                                     \
+    else return set_error(qs::QS_ERR_INVALID, "dtype must be QS_DTYPE_BF16 or QS_DTYPE_F32"); \
+  } while (0)
+
+extern "C" {
+
+int qs_hyb_state_space_prep_floats(int heads, int groups, int state_n, int vdim) { return hyb::ssd_row_floats(heads, groups, state_n, vdim); }
+
+int qs_hyb_state_space(void* out, int64_t out_stride, float* prep, float* o_raw, const void* proj, int64_t stride, const float* conv_w,
+                       const float* conv_b, float* conv_state, float* state, const float* a_log, const float* dt_bias, const float* skip,
+                       const float* norm_w, int norm_groups, float out_scale, const int32_t* tok_entry, const int32_t* tok_pos,
+                       const int32_t* entry_start, const int32_t* entry_len, const int32_t* entry_slot, const int32_t* entry_pos0, int tokens_n,
+                       int entries, int heads, int groups, int state_n, int vdim, int taps, float eps, int dtype, void* stream) {
+  QS_REQUIRE(out && prep && o_raw && proj && conv_w && state && a_log && dt_bias && skip && norm_w, "hyb_state_space: null tensor");
+  QS_REQUIRE(tok_entry && tok_pos && entry_start && entry_len && entry_slot && entry_pos0, "hyb_state_space: null batch table");
+  QS_REQUIRE(heads > 0 && groups > 0 && heads % groups == 0 && vdim > 0 && state_n > 0 && state_n <= 512, "hyb_state_space: groups divide heads, 0 < state <= 512");
+  QS_REQUIRE(taps >= 1 && taps <= kMaxTaps && (taps == 1 || conv_state != nullptr), "hyb_state_space: 1..17 convolution taps");
+  QS_REQUIRE(norm_groups > 0 && (heads * vdim) % norm_groups == 0 && (heads * vdim) / norm_groups <= 51200, "hyb_state_space: norm groups divide the row");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  QS_DT(dtype,
+        return launch_state_space<__nv_bfloat16>(out, out_stride, prep, o_raw, proj, stride, conv_w, conv_b, conv_state, state, a_log, dt_bias, skip, norm_w,
+                                                 norm_groups, out_scale, tok_entry, tok_pos, entry_start, entry_len, entry_slot, entry_pos0, tokens_n,
+                                                 entries, heads, groups, state_n, vdim, taps, eps, s),
+        return launch_state_space<float>(out, out_stride, prep, o_raw, proj, stride, conv_w, conv_b, conv_state, state, a_log, dt_bias, skip, norm_w,
+                                         norm_groups, out_scale, tok_entry, tok_pos, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries,
+                                         heads, groups, state_n, vdim, taps, eps, s));
+}
+
+int qs_hyb_lru_conv(void* u, const void* proj, int64_t stride, const float* x_bias, const float* conv_w, const float* conv_b, float* conv_state,
+                    const int32_t* tok_entry, const int32_t* tok_pos, const int32_t* entry_start, const int32_t* entry_len, const int32_t* entry_slot,
+                    const int32_t* entry_pos0, int tokens_n, int entries, int width, int taps, int dtype, void* stream) {
+  QS_REQUIRE(u && proj && conv_w, "hyb_lru_conv: null tensor");
+  QS_REQUIRE(tok_entry && tok_pos && entry_start && entry_len && entry_slot && entry_pos0, "hyb_lru_conv: null batch table");
+  QS_REQUIRE(width > 0 && taps >= 1 && taps <= kMaxTaps && (taps == 1 || conv_state != nullptr), "hyb_lru_conv: 1..17 convolution taps");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  QS_DT(dtype,
+        return launch_lru_conv<__nv_bfloat16>(u, proj, stride, x_bias, conv_w, conv_b, conv_state, tok_entry, tok_pos, entry_start, entry_len, entry_slot,
+                                              entry_pos0, tokens_n, entries, width, taps, s),
+        return launch_lru_conv<float>(u, proj, stride, x_bias, conv_w, conv_b, conv_state, tok_entry, tok_pos, entry_start, entry_len, entry_slot,
+                                      entry_pos0, tokens_n, entries, width, taps, s));
+}
+
+int qs_hyb_lru_scan(void* out, int64_t out_stride, float* state, float* sums, const void* u, const float* z, const void* proj, int64_t stride,
+                    const float* y_bias, const float* r_bias, const float* i_bias, const float* rate, const int32_t* tile_entry, const int32_t* tile_row0,
+                    int n_tiles, int n_short, const int32_t* entry_start, const int32_t* entry_len, const int32_t* entry_slot, const int32_t* entry_pos0,
+                    int tokens_n, int entries, int width, int blocks, int tile_rows, int long_min, int dtype, void* stream) {
+  QS_REQUIRE(out && state && u && z && proj && y_bias && r_bias && i_bias && rate, "hyb_lru_scan: null tensor");
+  QS_REQUIRE(entry_start && entry_len && entry_slot && entry_pos0, "hyb_lru_scan: null batch table");
+  QS_REQUIRE(n_tiles == 0 || (tile_entry && tile_row0 && sums && tile_rows > 0), "hyb_lru_scan: null tile table");
+  QS_REQUIRE(width > 0 && blocks > 0 && width % blocks == 0 && long_min > 0, "hyb_lru_scan: blocks divide the width");
+  if (tokens_n == 0) return qs::QS_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  QS_DT(dtype,
+        return launch_lru_scan<__nv_bfloat16>(out, out_stride, state, sums, u, z, proj, stride, y_bias, r_bias, i_bias, rate, tile_entry, tile_row0, n_tiles,
+                                              n_short, entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, width, blocks, tile_rows,
+                                              long_min, s),
+        return launch_lru_scan<float>(out, out_stride, state, sums, u, z, proj, stride, y_bias, r_bias, i_bias, rate, tile_entry, tile_row0, n_tiles, n_short,
+                                      entry_start, entry_len, entry_slot, entry_pos0, tokens_n, entries, width, blocks, tile_rows, long_min, s));
+}
+
+}  // extern "C"

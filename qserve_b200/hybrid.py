@@ -25,13 +25,15 @@ import ctypes
 
 from ._lib import AttnExtra, check, lib
 from .cache import HybridCache
-from .modelcfg import (AttentionMixerConfig, DeltaMixerConfig, GatedLinearMixerConfig, GateRecurrenceMixerConfig, HybridConfig,
-                       LatentAttentionMixerConfig, MlpConfig, MoeConfig, ParallelMixerConfig, RetentionMixerConfig)
+from .modelcfg import (AttentionMixerConfig, DeltaMixerConfig, GatedLinearMixerConfig, GatedUnitMixerConfig, GateRecurrenceMixerConfig,
+                       HybridConfig, LatentAttentionMixerConfig, MlpConfig, MoeConfig, ParallelMixerConfig, RetentionMixerConfig,
+                       StateSpaceMixerConfig)
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 _NORM_KIND = {"rms": 1, "layer": 2}      # QS_NORM_RMS, QS_NORM_LAYER
 _ROUTER_MODE = {"softmax": 0, "sigmoid": 1}  # QS_ROUTER_SOFTMAX, QS_ROUTER_SIGMOID_GROUPS
 _ACT = {"gelu_tanh": 0, "silu": 1}           # QS_ACT_GELU_TANH, QS_ACT_SILU
+_PLAIN_ACT = ("gelu_tanh", "relu2")          # dense feed-forwards without a gate
 _ROT_LAYOUT = {"interleaved": 0, "half": 1}
 _F32_OUT = [None]  # whether torch.mm takes out_dtype on this build (found at first use)
 
@@ -52,6 +54,18 @@ def _mm_f32(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
         except RuntimeError:  # a shape or stride this form of the product does not take
             pass
     return torch.mm(a, b).float()
+
+
+def _bmm_f32(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+    """Batched a @ b with an fp32 result; where the library does not offer that for 16-bit operands, the product of their fp32 copies."""
+    if a.dtype == torch.float32:
+        return torch.bmm(a, b)
+    if _F32_OUT[0] is not False:
+        try:
+            return torch.bmm(a, b, out_dtype=torch.float32)
+        except (TypeError, RuntimeError):
+            pass
+    return torch.bmm(a.float(), b.float())
 
 
 def _pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
@@ -195,7 +209,8 @@ class MultiMapAttentionMixer(_Mixer):
     o = a1 - lambda a2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, then unit RMS per head and a factor (1 - diff).
     With one map: optional projection biases, unit-RMS q / k (with gains shared by the heads), a learned temperature per head (folded into the
     prepared query), a sink term in the denominator, a mask by chunks of positions and / or a window that may keep the sequence's first
-    positions visible, a tanh cap on the scores, a linear distance bias per head, values tied to the key projection's raw output (no value
+    positions visible, q and k normed as whole rows ahead of the split into heads with queries that grow with the logarithm of the position, a
+    tanh cap on the scores, a linear distance bias per head, values tied to the key projection's raw output (no value
     projection) or brought to unit RMS per head before they are cached, an output bias, and a sigmoid gate per head or per output number (its
     logits are the last columns of the mixer's projection rows)."""
 
@@ -203,7 +218,8 @@ class MultiMapAttentionMixer(_Mixer):
         self.m, self.eps = m, eps
         assert m.heads % m.kv_heads == 0
         f32 = lambda t: t.to(torch.float32).to(device).contiguous()
-        self.general = m.rot is None or m.rot.layout != "interleaved" or m.bias or m.qk_norm or m.head_temp or m.tied_values or m.value_norm
+        self.general = m.rot is None or m.rot.layout != "interleaved" or m.bias or m.qk_norm or m.head_temp or m.tied_values or m.value_norm or \
+            m.row_norm
         plus = m.sink or m.keep_first or m.distance_slope > 0.0 or m.head_gate or m.qk_gain or m.gate_wide or m.softcap > 0.0 or m.sink_score is not None
         if (self.general or plus) and m.maps != 1:
             raise ValueError("biases, unit-RMS q / k / v, head temperatures, sinks, kept first positions, score caps, distance biases, tied values, "
@@ -218,9 +234,15 @@ class MultiMapAttentionMixer(_Mixer):
             raise ValueError("values tied to the keys need vdim == dim")
         if m.qk_gain and not m.qk_norm:
             raise ValueError("q / k gains belong to the unit-RMS q / k")
+        if m.row_norm and (m.rot is not None or m.qk_norm or m.qk_gain or m.head_temp or m.tied_values or m.value_norm):
+            raise ValueError("row norms of q / k go without rotations, norms and temperatures per head, tied values and value norms")
+        if m.temp_coef != 0.0 and not (m.row_norm and m.temp_every > 0.0):
+            raise ValueError("a query temperature by position goes with row norms of q / k")
         parts = ["q", "k"] + ([] if m.tied_values else ["v"])
         self.bias = f32(torch.cat([w[n + ".b"] for n in parts], 0)) if m.bias else None
-        self.q_gain, self.k_gain = (f32(w["q.norm"]), f32(w["k.norm"])) if m.qk_gain else (None, None)
+        self.q_gain, self.k_gain = (f32(w["q.norm"]), f32(w["k.norm"])) if m.qk_gain or m.row_norm else (None, None)
+        if m.row_norm and (self.q_gain.numel() != m.heads * m.dim or self.k_gain.numel() != m.kv_heads * m.dim):
+            raise ValueError("q / k gains of row norms have heads * dim and kv_heads * dim numbers")
         if m.qk_gain and (self.q_gain.numel() != m.dim or self.k_gain.numel() != m.dim):
             raise ValueError("q / k gains have `dim` numbers")
         sl = m.slopes()
@@ -271,7 +293,12 @@ class MultiMapAttentionMixer(_Mixer):
         if self.extra:
             gate = proj.data_ptr() + self.col_g * proj.element_size() if self.gated else None
             extra = ctypes.byref(AttnExtra(m.keep_first, _p(self.slopes), gate, proj.stride(0), 1 if m.gate_wide else 0, m.softcap))
-        if self.general:
+        if m.row_norm:
+            check(lib.qs_hyb_qk_row_norm_append(proj.data_ptr(), proj.stride(0), _p(self.bias), self.q_gain.data_ptr(), self.k_gain.data_ptr(), m.temp_coef,
+                                                m.temp_every, _p(b.tok_slot), _p(b.tok_pos), _p(b.block_table), b.block_table.shape[1],
+                                                run_cache["k"].data_ptr(), run_cache["v"].data_ptr(), self.eps, b.n_tokens, m.heads * m.dim,
+                                                m.kv_heads * m.dim, m.kv_heads * m.vdim, page_size, dt, stream))
+        elif self.general:
             check(lib.qs_hyb_qk_prepare_append(proj.data_ptr(), proj.stride(0), _p(self.bias), _p(self.temp), _p(b.tok_slot), _p(b.tok_pos),
                                                _p(b.block_table), b.block_table.shape[1], run_cache["k"].data_ptr(), run_cache["v"].data_ptr(),
                                                _p(self.inv_freq), 1 if m.rot is not None and m.rot.layout == "half" else 0,
@@ -546,9 +573,89 @@ class LatentAttentionMixer(_Mixer):
 LATENT_IMPL = None  # tests: "plain" keeps the latent attention on the CUDA-core kernel, "latent" keeps prompt portions on the latent-space tiles
 
 
+class StateSpaceMixer(_Mixer):
+    """Mamba-2: [z | x | B | C | dt] = W_in h; x, B, C pass a short causal convolution and silu; per head S <- exp(-exp(A_log) dt) S + dt B x^T,
+    y = S^T C + D x with dt = softplus(dt + dt_bias); y silu(z) in unit-RMS parts times a gain.  The fp32 state and the convolution's last inputs
+    live in the sequence's slot."""
+
+    def __init__(self, m: StateSpaceMixerConfig, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.m, self.eps = m, eps
+        inner, channels = m.heads * m.vdim, m.heads * m.vdim + 2 * m.groups * m.state
+        if w["in"].shape[0] != inner + channels + m.heads:
+            raise ValueError(f"state space weight in: {tuple(w['in'].shape)} does not have {inner + channels + m.heads} rows")
+        self.w_in = _pad_rows(w["in"]).to(device=device, dtype=dtype).contiguous()
+        self.in_features, self.out_features = self.w_in.shape[0], inner
+        self.w_out = w["o"]
+        f32 = lambda t: t.to(torch.float32).to(device).contiguous()
+        self.conv_w, self.conv_b = f32(w["conv"]), f32(w["conv.b"])
+        self.a_log, self.dt_bias, self.skip, self.norm_w = f32(w["A_log"]), f32(w["dt_bias"]), f32(w["D"]), f32(w["norm"])
+        if tuple(self.conv_w.shape) != (channels, m.conv) or self.conv_b.numel() != channels:
+            raise ValueError("state space: the convolution is [heads * vdim + 2 groups * state, conv] with a bias per channel")
+        if any(t.numel() != m.heads for t in (self.a_log, self.dt_bias, self.skip)) or self.norm_w.numel() != inner:
+            raise ValueError("state space: A_log, dt_bias and D have one number per head, norm has heads * vdim")
+        self.prep_width = int(lib.qs_hyb_state_space_prep_floats(m.heads, m.groups, m.state, m.vdim))
+        self.out_scale = 1.0
+
+    def scratch_floats(self, tokens: int) -> int:
+        return tokens * (self.prep_width + self.out_features)
+
+    def run(self, proj, out, b: StepBatch, run_cache: dict, page_size: int, scratch: torch.Tensor, dt: int, stream) -> None:
+        m, T = self.m, b.n_tokens
+        prep = scratch[: T * self.prep_width]
+        o_raw = scratch[T * self.prep_width: T * (self.prep_width + self.out_features)]
+        check(lib.qs_hyb_state_space(out.data_ptr(), out.stride(0), prep.data_ptr(), o_raw.data_ptr(), proj.data_ptr(), proj.stride(0),
+                                     self.conv_w.data_ptr(), self.conv_b.data_ptr(), run_cache["conv"].data_ptr(), run_cache["state"].data_ptr(),
+                                     self.a_log.data_ptr(), self.dt_bias.data_ptr(), self.skip.data_ptr(), self.norm_w.data_ptr(), m.norm_groups,
+                                     self.out_scale, _p(b.tok_entry), _p(b.tok_pos), _p(b.entry_start), _p(b.entry_len), _p(b.entry_slot),
+                                     _p(b.entry_pos0), T, b.n_entries, m.heads, m.groups, m.state, m.vdim, m.conv, self.eps, dt, stream))
+
+
+class GatedUnitMixer(_Mixer):
+    """Griffin's recurrent block: y = gelu_tanh(W_y h + b), u = conv(W_x h + b); gates r, i = sigmoid of block-diagonal projections of u (one
+    batched product, fp32 logits); log a = -rate r softplus(lam), S <- a S + sqrt(1 - a^2) i u per channel, output S y.  The fp32 state and
+    the convolution's last inputs live in the sequence's slot."""
+
+    def __init__(self, m: GatedUnitMixerConfig, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.m, W, nb = m, m.width, m.blocks
+        wb = W // nb
+        for name, shape in (("ra", (nb, wb, wb)), ("ri", (nb, wb, wb)), ("conv", (W, m.conv))):
+            if tuple(w[name].shape) != shape:
+                raise ValueError(f"gated unit weight {name}: {tuple(w[name].shape)} is not {shape}")
+        for name in ("y.b", "x.b", "conv.b", "ra.b", "ri.b", "lam"):
+            if w[name].numel() != W:
+                raise ValueError(f"gated unit weight {name} does not have {W} numbers")
+        if w["y"].shape[0] != W or w["x"].shape[0] != W:
+            raise ValueError(f"gated unit weights y and x have {W} rows")
+        self.w_in = _pad_rows(torch.cat([w["y"], w["x"]], 0)).to(device=device, dtype=dtype).contiguous()
+        self.in_features, self.out_features = self.w_in.shape[0], W
+        self.w_gates = torch.cat([w["ra"], w["ri"]], 1).to(device=device, dtype=dtype).contiguous()  # [blocks, 2 W / blocks, W / blocks]
+        self.w_out = w["o"]
+        f32 = lambda t: t.to(torch.float32).reshape(-1).to(device).contiguous()
+        self.y_bias, self.x_bias, self.conv_b, self.r_bias, self.i_bias = (f32(w[n]) for n in ("y.b", "x.b", "conv.b", "ra.b", "ri.b"))
+        self.conv_w = w["conv"].to(torch.float32).to(device).contiguous()
+        self.rate = f32(-m.decay_rate * torch.nn.functional.softplus(w["lam"].double(), threshold=1e9))
+
+    def scratch_floats(self, tokens: int) -> int:
+        return max(1, tokens // StepBatch.TILE_MIN) * 2 * self.m.width  # at most one tile of a long entry per TILE_MIN tokens
+
+    def run(self, proj, out, b: StepBatch, run_cache: dict, page_size: int, scratch: torch.Tensor, dt: int, stream) -> None:
+        m, T = self.m, b.n_tokens
+        u = torch.empty((T, m.width), dtype=proj.dtype, device=proj.device)
+        tables = (_p(b.entry_start), _p(b.entry_len), _p(b.entry_slot), _p(b.entry_pos0))
+        check(lib.qs_hyb_lru_conv(u.data_ptr(), proj.data_ptr(), proj.stride(0), self.x_bias.data_ptr(), self.conv_w.data_ptr(), self.conv_b.data_ptr(),
+                                  run_cache["conv"].data_ptr(), _p(b.tok_entry), _p(b.tok_pos), *tables, T, b.n_entries, m.width, m.conv, dt, stream))
+        z = _bmm_f32(u.view(T, m.blocks, -1).transpose(0, 1), self.w_gates.transpose(1, 2))  # [blocks, T, 2 W / blocks]
+        check(lib.qs_hyb_lru_scan(out.data_ptr(), out.stride(0), run_cache["state"].data_ptr(), scratch.data_ptr(), u.data_ptr(), z.data_ptr(),
+                                  proj.data_ptr(), proj.stride(0), self.y_bias.data_ptr(), self.r_bias.data_ptr(), self.i_bias.data_ptr(),
+                                  self.rate.data_ptr(), _p(b.tile_entry), _p(b.tile_row0), b.n_tiles, b.n_short, *tables, T, b.n_entries, m.width, m.blocks,
+                                  StepBatch.TILE_ROWS, StepBatch.TILE_MIN, dt, stream))
+
+
 class ParallelMixer(_Mixer):
-    """Two mixers on the same input: one product makes both projection rows, each runs on its part, and the result is
-    scale (norm(W_o,left heads_left) gain_left + norm(W_o,right heads_right) gain_right) with plain RMS norms over the width."""
+    """Two mixers on the same input: one product makes both projection rows and each runs on its part.  With branch norms the result is
+    scale (norm(W_o,left heads_left) gain_left + norm(W_o,right heads_right) gain_right) with plain RMS norms over the width.  Without, it is
+    left_scale W_o,left heads_left + right_scale W_o,right heads_right: the factors ride in the mixers' own last kernels and ONE product
+    [heads_left | heads_right] @ [W_o,left | W_o,right]^T sums the branches in its fp32 accumulation."""
 
     def __init__(self, m: ParallelMixerConfig, w: Dict[str, torch.Tensor], eps: float, dtype, device):
         self.m, self.eps = m, eps
@@ -560,12 +667,24 @@ class ParallelMixer(_Mixer):
         self.w_in = torch.cat([self.left.w_in, self.right.w_in], 0).contiguous()
         del self.left.w_in, self.right.w_in
         f32 = lambda t: t.to(torch.float32).to(device).contiguous()
-        self.gain_left, self.gain_right = f32(w["left.out"]), f32(w["right.out"])
+        if m.branch_norm:
+            self.gain_left, self.gain_right = f32(w["left.out"]), f32(w["right.out"])
+            return
+        if not hasattr(self.left, "out_scale") or not hasattr(self.right, "out_scale"):
+            raise NotImplementedError("a weighted sum of side-by-side mixers whose last kernels take no factor")
+        if self.left.out_bias is not None or self.right.out_bias is not None:
+            raise NotImplementedError("a weighted sum of side-by-side mixers with output biases")
+        self.left.out_scale *= m.left_scale
+        self.right.out_scale *= m.right_scale
+        self.w_out = torch.cat([self.left.w_out, self.right.w_out], 1)
+        del self.left.w_out, self.right.w_out
 
     def scratch_floats(self, tokens: int) -> int:
         return max(self.left.scratch_floats(tokens), self.right.scratch_floats(tokens))  # they run one after the other
 
     def place_out(self, st) -> None:
+        if not self.m.branch_norm:
+            return super().place_out(st)
         self.left.place_out(st)
         self.right.place_out(st)
 
@@ -575,6 +694,8 @@ class ParallelMixer(_Mixer):
         self.right.run(proj[:, a:], out[:, oa:], b, run_cache["right"], page_size, scratch, dt, stream)
 
     def project(self, cat: torch.Tensor, dt: int, stream, f32: bool = False):
+        if not self.m.branch_norm:
+            return super().project(cat, dt, stream, f32)
         oa = self.left.out_features
         yl, fl = self.left.project(cat[:, :oa], dt, stream)
         yr, fr = self.right.project(cat[:, oa:], dt, stream)
@@ -589,7 +710,7 @@ class ParallelMixer(_Mixer):
 
 MIXERS = {AttentionMixerConfig: MultiMapAttentionMixer, DeltaMixerConfig: GatedDeltaMixer, GateRecurrenceMixerConfig: GateRecurrenceMixer,
           RetentionMixerConfig: RetentionMixer, ParallelMixerConfig: ParallelMixer, LatentAttentionMixerConfig: LatentAttentionMixer,
-          GatedLinearMixerConfig: GatedLinearMixer}
+          GatedLinearMixerConfig: GatedLinearMixer, StateSpaceMixerConfig: StateSpaceMixer, GatedUnitMixerConfig: GatedUnitMixer}
 
 
 # ------------------------------------------------------------------------------------------------------------------------
@@ -651,7 +772,7 @@ class MoeFeedForward:
         top_idx = torch.empty((T, c.top), dtype=torch.int32, device=dev)
         top_w = torch.empty((T, c.top), dtype=torch.float32, device=dev)
         check(lib.qs_hyb_moe_router(route.data_ptr(), top_idx.data_ptr(), top_w.data_ptr(), h.data_ptr(), self.w_router.data_ptr(), T, W, c.experts,
-                                    c.top, _ROUTER_MODE[c.router], _p(self.correction), c.groups, c.keep, dt, stream))
+                                    c.top, _ROUTER_MODE[c.router], _p(self.correction), c.groups, c.keep, 1 if c.renormalize else 0, c.weight_scale, dt, stream))
         if self.impl == "dense":
             gu = torch.mm(h, self.w_in.t())
             act = torch.empty((T, self.F), dtype=h.dtype, device=dev)
@@ -682,33 +803,36 @@ class MoeFeedForward:
 
 
 class DenseFeedForward:
-    """W_down (act(W_gate h + b_gate) * (W_up h + b_up)) [+ b_down], act gelu_tanh or silu.  The down projection's bias (`out_bias`) is left
+    """W_down (act(W_gate h + b_gate) * (W_up h + b_up)) [+ b_down], act gelu_tanh or silu; without a gate W_down act(W_up h + b_up) [+ b_down], act
+    gelu_tanh or the square of relu.  The down projection's bias (`out_bias`) is left
     to the block, which adds it where it takes the rows."""
 
     def __init__(self, c: MlpConfig, w: Dict[str, torch.Tensor], width: int, dtype, device):
         st = lambda t: t.to(device=device, dtype=dtype).contiguous()
-        if not c.gated:
-            raise NotImplementedError("a dense feed-forward without a gate, outside a parallel block")
-        if c.act not in _ACT:
-            raise ValueError(f"unknown activation {c.act!r}")
-        if tuple(w["gate"].shape) != (c.ff, width) or tuple(w["up"].shape) != (c.ff, width) or tuple(w["down"].shape) != (width, c.ff):
+        if c.act not in (_ACT if c.gated else _PLAIN_ACT):
+            raise ValueError(f"unknown activation {c.act!r} (gated: {c.gated})")
+        ins = ("gate", "up") if c.gated else ("up",)
+        if any(tuple(w[n].shape) != (c.ff, width) for n in ins) or tuple(w["up"].shape) != (c.ff, width) or tuple(w["down"].shape) != (width, c.ff):
             raise ValueError("dense feed-forward: the projections do not match ff x width")
-        self.ff, self.act = c.ff, _ACT[c.act]
-        self.w_in, self.w_down = st(torch.cat([w["gate"], w["up"]], 0)), st(w["down"])
+        self.ff, self.act, self.gated = c.ff, _ACT[c.act] if c.gated else c.act, c.gated
+        self.w_in, self.w_down = st(torch.cat([w[n] for n in ins], 0)), st(w["down"])
         self.in_bias = self.out_bias = None
         if c.bias:
-            self.in_bias = torch.cat([w["gate.b"], w["up.b"]], 0).to(torch.float32).to(device).contiguous()
+            self.in_bias = torch.cat([w[n + ".b"] for n in ins], 0).to(torch.float32).to(device).contiguous()
             self.out_bias = w["down.b"].to(torch.float32).to(device).contiguous()
-            if self.in_bias.numel() != 2 * c.ff or self.out_bias.numel() != width:
+            if self.in_bias.numel() != len(ins) * c.ff or self.out_bias.numel() != width:
                 raise ValueError("dense feed-forward: the biases do not match their projections")
 
     def run(self, h: torch.Tensor, dt: int, stream):
         return self.finish(torch.mm(h, self.w_in.t()), dt, stream)
 
     def finish(self, gu: torch.Tensor, dt: int, stream):
-        """From the rows [gate | up (| columns of somebody else)] of the input product on."""
+        """From the rows [gate | up (| columns of somebody else)], or [up (| ...)] without a gate, of the input product on."""
         act = torch.empty((gu.shape[0], self.ff), dtype=gu.dtype, device=gu.device)
-        if self.in_bias is None and self.act == 0 and gu.stride(0) == 2 * self.ff:
+        if not self.gated:
+            kernel = lib.qs_hyb_bias_relu_squared if self.act == "relu2" else lib.qs_hyb_bias_gelu_tanh
+            check(kernel(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), _p(self.in_bias), gu.shape[0], self.ff, dt, stream))
+        elif self.in_bias is None and self.act == 0 and gu.stride(0) == 2 * self.ff:
             check(lib.qs_hyb_gelu_tanh_mul(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.shape[0], self.ff, dt, stream))
         else:
             check(lib.qs_hyb_bias_gated_act(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), _p(self.in_bias), gu.shape[0], self.ff, self.act, dt,
@@ -774,13 +898,14 @@ class HybridDecoder:
         st = lambda t: t.to(device=dev, dtype=dtype).contiguous()
         f32 = lambda t: t.to(torch.float32).to(dev).contiguous()
         W = cfg.width
-        if tuple(weights["embed"].shape) != (cfg.vocab, W) or tuple(weights["head"].shape) != (cfg.vocab, W):
+        head = weights["embed" if cfg.tied_head else "head"]
+        if tuple(weights["embed"].shape) != (cfg.vocab, W) or tuple(head.shape) != (cfg.vocab, W):
             raise ValueError("embed / head do not match vocab x width")
         self.embed = st(weights["embed"])
         self.pair = st(weights["bigram"]) if cfg.pair_buckets > 0 else None
         if self.pair is not None and self.pair.shape[0] != cfg.pair_buckets + 1:
             raise ValueError("the pair table must have buckets + 1 rows")
-        self.head = st(weights["head"])
+        self.head = self.embed if cfg.tied_head else st(head)
         # a factor on the logits rides in the last norm's gain
         self.final_norm = f32(weights["final.norm"])
         if cfg.logit_scale != 1.0:
@@ -790,10 +915,14 @@ class HybridDecoder:
             raise ValueError(f"unknown block form {cfg.block!r}")
         if cfg.block != "sandwich" and (cfg.residual_gate or cfg.embed_norm or cfg.residual_mult != 1.0):
             raise NotImplementedError("residual gates, a residual factor and a normed embedding are built for sandwich blocks")
+        if cfg.loop_add and (cfg.block != "sequential" or cfg.streams > 0 or cfg.norm_groups != 1 or cfg.norm_offset != 0.0):
+            raise NotImplementedError("a loop whose passes add the embedding output is built for sequential blocks on one stream with plain norms")
         if cfg.norm_groups < 1 or W % cfg.norm_groups:
             raise ValueError("norm groups must divide the width")
         self.embed_norm = f32(weights["embed.norm"]) if cfg.embed_norm else None
         self.n_streams = max(cfg.streams, 1) if cfg.block == "sequential" else 1
+        # sequential blocks on one stream with plain gains: fp32 sublayer rows land in the stream inside the next norm kernel
+        self.one_stream = cfg.block == "sequential" and cfg.streams <= 0 and cfg.norm_groups == 1 and cfg.norm_offset == 0.0
         one = torch.ones(1, dtype=torch.float32, device=dev)
 
         def hyper(pre: str) -> _Hyper:
@@ -834,7 +963,7 @@ class HybridDecoder:
                 if ly.mlp is not None:
                     fw = {k[len(pre) + 4:]: v for k, v in weights.items() if k.startswith(pre + "mlp.")}
                     ff = FEED_FORWARDS[type(ly.mlp)](ly.mlp, fw, W, dtype, dev)
-                    if getattr(ff, "out_bias", None) is not None:
+                    if getattr(ff, "out_bias", None) is not None and not self.one_stream:
                         raise NotImplementedError("a biased dense feed-forward on hyper-connected streams")
                     norm2, hc2 = f32(weights[pre + "norm2"]), hyper(pre + "hc2.")
                 self.layers.append(_Layer(mixer, f32(weights[pre + "norm1"]), norm2, None, None, ff, hyper(pre + "hc1."), hc2))
@@ -842,6 +971,8 @@ class HybridDecoder:
             outs = [mixer.w_out]
             w_mlp_in, norm2, ff = None, None, 0
             dense = isinstance(ly.mlp, MlpConfig)
+            if dense and ly.mlp.act != "gelu_tanh":
+                raise NotImplementedError("parallel blocks fold gelu_tanh feed-forwards")
             if dense:  # folded: its activation sits beside the mixer's heads as input of ONE output product
                 ff = ly.mlp.ff
                 w_mlp_in = st(torch.cat([weights[pre + "mlp.gate"], weights[pre + "mlp.up"]], 0) if ly.mlp.gated else weights[pre + "mlp.up"])
@@ -951,6 +1082,8 @@ class HybridDecoder:
                 self._scratch = torch.empty(need, dtype=torch.float32, device=dev)
             scratch = self._scratch
         if cfg.block == "sequential":
+            if self.one_stream:
+                return self._forward_one_stream(x.view(T, W), b, cache, tap, scratch, s)
             return self._forward_sequential(x, b, cache, tap, scratch, s)
         if cfg.block == "post":
             return self._forward_post(x, b, cache, tap, scratch, s)
@@ -1049,6 +1182,35 @@ class HybridDecoder:
         self._stream_norm(None, total, x, pending, None, None, s)
         return total
 
+    def _forward_one_stream(self, x, b: StepBatch, cache: HybridCache, tap, scratch, s) -> torch.Tensor:
+        """Sequential blocks on a plain residual stream: every sublayer's rows (the output product's fp32 accumulators) wait as `pending` and land
+        inside the next norm kernel; at the start of a later pass of the loop the embedding output lands with them."""
+        cfg, dev, dt, T, W = self.cfg, self.device, self.dt, b.n_tokens, self.cfg.width
+        again = set(cfg.pass_starts()[1:]) if cfg.loop_add else set()
+        x0 = x.clone() if again else None
+        pending = None
+        h = torch.empty((T, W), dtype=self.dtype, device=dev)
+        for run, li in enumerate(self.schedule):
+            ly = self.layers[li]
+            if run in again:
+                y, y32, _, _, yb = pending if pending is not None else (None, False, None, False, None)
+                pending = (y, y32, x0, True, yb)
+            self._land(x, pending, s, out_h=h, w=ly.norm1)
+            proj = torch.mm(h, ly.mixer.w_in.t())
+            cat = torch.empty((T, ly.mixer.out_features), dtype=self.dtype, device=dev)
+            ly.mixer.run(proj, cat, b, cache.runs[run], cache.page_size, scratch, dt, s)
+            pending = (*ly.mixer.project(cat, dt, s, f32=True), None, False, None)
+            if ly.ff is not None:
+                self._land(x, pending, s, out_h=h, w=ly.norm2)
+                pending = (*ly.ff.run(h, dt, s), None, False, getattr(ly.ff, "out_bias", None))
+            if tap is not None:  # observers want the stream after every run
+                self._land(x, pending, s)
+                pending = None
+                tap(run, x)
+        if pending is not None:
+            self._land(x, pending, s)
+        return x
+
     def _forward_post(self, x, b: StepBatch, cache: HybridCache, tap, scratch, s) -> torch.Tensor:
         cfg, dev, dt, T, W = self.cfg, self.device, self.dt, b.n_tokens, self.cfg.width
         # the sublayers' input: the fp32 stream as it is with fp32 storage, else its storage-type copy, which every landing kernel renews
@@ -1123,7 +1285,7 @@ class HybridDecoder:
                                       W, self.dt, s))
         else:
             self._land(x_rows, None, s, out_h=h, w=self.final_norm, bias=self.final_norm_b)
-        out = _mm_f32(h, self.head.t()) if self.cfg.logit_softcap > 0.0 or self.cfg.block in ("post", "sandwich") else torch.mm(h, self.head.t()).float()
+        out = _mm_f32(h, self.head.t()) if self.cfg.logit_softcap > 0.0 or self.cfg.block in ("post", "sandwich") or self.one_stream else torch.mm(h, self.head.t()).float()
         if self.cfg.logit_softcap > 0.0:
             check(lib.qs_hyb_softcap(out.data_ptr(), out.numel(), self.cfg.logit_softcap, s))
         return out
@@ -1143,7 +1305,23 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
         if isinstance(m, ParallelMixerConfig):
             mixer_weights(p + "left.", m.left)
             mixer_weights(p + "right.", m.right)
+            if not m.branch_norm:
+                return
             w[p + "left.out"], w[p + "right.out"] = 1.0 + r(W, s=0.1), 1.0 + r(W, s=0.1)
+            return
+        if isinstance(m, StateSpaceMixerConfig):
+            inner, gn = m.heads * m.vdim, m.groups * m.state
+            w[p + "in"], w[p + "conv"], w[p + "conv.b"] = r(2 * inner + 2 * gn + m.heads, W, s=W ** -0.5), r(inner + 2 * gn, m.conv, s=0.5), r(inner + 2 * gn, s=0.1)
+            w[p + "dt_bias"], w[p + "A_log"], w[p + "D"] = r(m.heads, s=0.5) - 2.0, r(m.heads, s=0.5), 1.0 + r(m.heads, s=0.1)
+            w[p + "norm"], w[p + "o"] = 1.0 + r(inner, s=0.1), r(W, inner, s=inner ** -0.5)
+            return
+        if isinstance(m, GatedUnitMixerConfig):
+            R, wb = m.width, m.width // m.blocks
+            w[p + "y"], w[p + "x"], w[p + "y.b"], w[p + "x.b"] = r(R, W, s=W ** -0.5), r(R, W, s=W ** -0.5), r(R, s=0.1), r(R, s=0.1)
+            w[p + "conv"], w[p + "conv.b"], w[p + "lam"] = r(R, m.conv, s=0.5), r(R, s=0.1), r(R, s=0.5) - 2.0
+            for n in ("ra", "ri"):
+                w[p + n], w[p + n + ".b"] = r(m.blocks, wb, wb, s=wb ** -0.5), r(m.blocks, wb, s=0.1)
+            w[p + "o"] = r(W, R, s=R ** -0.5)
             return
         H, D, Dv = m.heads, m.dim, m.vdim
         if isinstance(m, LatentAttentionMixerConfig):
@@ -1169,6 +1347,8 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
                 w[p + "v"] = r(G * Dv, W, s=W ** -0.5)
             if m.qk_gain:
                 w[p + "q.norm"], w[p + "k.norm"] = 1.0 + r(D, s=0.1), 1.0 + r(D, s=0.1)
+            if m.row_norm:
+                w[p + "q.norm"], w[p + "k.norm"] = 1.0 + r(H * D, s=0.1), 1.0 + r(G * D, s=0.1)
             if m.head_gate or m.gate_wide:
                 w[p + "g"] = r(H * Dv if m.gate_wide else H, W, s=W ** -0.5)
             if m.out_bias:
@@ -1203,7 +1383,10 @@ def random_weights(cfg: HybridConfig, seed: int = 0, device: Optional[torch.devi
         w[p + "o"] = r(W, H * Dv, s=(H * Dv) ** -0.5)
 
     gain = (lambda: 1.0 + r(W, s=0.1)) if cfg.norm_offset == 0.0 else (lambda: r(W, s=0.1))
-    w = {"embed": r(cfg.vocab, W), "head": r(cfg.vocab, W, s=W ** -0.5), "final.norm": gain()}
+    w = {"embed": r(cfg.vocab, W, s=W ** -0.5 if cfg.tied_head else 1.0)}
+    if not cfg.tied_head:
+        w["head"] = r(cfg.vocab, W, s=W ** -0.5)
+    w["final.norm"] = gain()
     layer_norm = cfg.norm_kind == "layer"
     if cfg.embed_norm:
         w["embed.norm"] = gain()

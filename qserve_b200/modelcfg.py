@@ -102,6 +102,9 @@ class AttentionMixerConfig:
     value_norm: bool = False  # value heads are brought to unit RMS before they are cached
     sink_score: Optional[float] = None  # the softmax denominator has one more term exp(sink_score) without a value, the same for every head
     out_bias: bool = False   # the output projection has a bias (tensor o.b)
+    row_norm: bool = False   # q and k are each brought to unit RMS as one row ahead of the split into heads, times gains of that size (tensors q.norm, k.norm)
+    temp_coef: float = 0.0   # with row_norm: the query at position p is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+    temp_every: float = 1.0
 
     def slopes(self):
         """Per-head slope of the distance bias (float64 list), or None."""
@@ -144,12 +147,39 @@ class GatedLinearMixerConfig:
 
 
 @dataclass(frozen=True)
+class StateSpaceMixerConfig:
+    """Mamba-2: per head a [state, vdim] fp32 state that decays by one number per (token, head) and takes the outer product of B and dt x; B and C
+    are shared by `groups` runs of heads.  x, B and C pass a short causal convolution of `conv` taps and silu.  The heads' outputs times silu of a
+    gate are brought to unit RMS in `norm_groups` equal parts."""
+    heads: int
+    state: int
+    vdim: int
+    groups: int
+    conv: int
+    norm_groups: int = 1
+
+
+@dataclass(frozen=True)
+class GatedUnitMixerConfig:
+    """Griffin's recurrent block: a real-gated linear recurrent unit (RG-LRU) of `width` channels behind a short causal convolution of `conv` taps,
+    times a gelu branch.  Its two gates are projections of the convolved row, block-diagonal in `blocks` equal parts; the logarithm of the
+    decay is -decay_rate * gate * softplus(lam)."""
+    width: int
+    blocks: int
+    conv: int
+    decay_rate: float = 8.0
+
+
+@dataclass(frozen=True)
 class ParallelMixerConfig:
-    """Two mixers side by side on the same input (tensors under left.* / right.*); each output is RMS-normed over the width with its own gain
-    (left.out / right.out), the result is `scale` times their sum."""
+    """Two mixers side by side on the same input (tensors under left.* / right.*).  branch_norm: each output is RMS-normed over the width with its
+    own gain (left.out / right.out), the result is `scale` times their sum.  Otherwise it is left_scale * left + right_scale * right."""
     left: object
     right: object
     scale: float = 0.5
+    branch_norm: bool = True
+    left_scale: float = 1.0
+    right_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -189,7 +219,7 @@ class LatentAttentionMixerConfig:
 @dataclass(frozen=True)
 class MlpConfig:
     """Dense feed-forward.  gated: W_down(act(W_gate h) * W_up h); not gated: W_down act(W_up h).  bias: every projection has one.
-    act: "gelu_tanh" or "silu"."""
+    act: "gelu_tanh", "silu" or "relu2" (the square of relu; not gated only)."""
     kind: str
     ff: int
     gated: bool = True
@@ -205,7 +235,8 @@ class MoeConfig:
     router "softmax": scores softmax over all experts, the winners weighted by their scores as they are.
     router "sigmoid": scores sigmoid(logit); the choice is made on score + a learned correction per expert (tensor `correction`), restricted
     to the `keep` best of `groups` equal groups of neighbouring experts (a group's score: the sum of its two largest choice scores); the
-    winners are weighted by their scores divided by the winners' sum."""
+    winners are weighted by their scores divided by the winners' sum (`renormalize`) or by their scores as they are.
+    weight_scale: a factor on every weight."""
     experts: int
     top: int
     ff: int
@@ -219,6 +250,8 @@ class MoeConfig:
     correction: bool = False
     groups: int = 1
     keep: int = 1
+    renormalize: bool = True
+    weight_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -256,6 +289,8 @@ class HybridConfig:
     residual_gate: bool = False  # "sandwich" blocks: a sublayer's output times sigmoid(W h + b) of its input h, ahead of its norm (tensors rg1, rg1.b, rg2, rg2.b)
     embed_norm: bool = False    # "sandwich" blocks: the embedding is normed (tensor embed.norm)
     logit_scale: float = 1.0    # logits <- logit_scale * head x, ahead of a cap
+    tied_head: bool = False     # the vocabulary projection is the embedding table as stored (no tensor head)
+    loop_add: bool = False      # before the first layer of every pass of the loop but the first: x <- x + x0 (x0 the embedding output)
     layer_scale: bool = False   # "post" blocks: a normed sublayer output is multiplied per channel by a learned row (tensors ls1, ls2)
 
     def schedule(self):
@@ -449,9 +484,55 @@ def parse_nagosun(c: dict) -> HybridConfig:
                         logit_scale=float(c.get("logit_scale", 1.0)))
 
 
+def parse_tumitar(c: dict) -> HybridConfig:
+    """Tumitar: sequential pre-norm blocks on one residual stream with plain gains, a scaled embedding that is also the vocabulary projection;
+    mixers `parallel` (a weighted sum of softmax attention with biases, q / k normed as whole rows, queries that grow with the position, a sink of
+    fixed score 0, and of a Mamba-2 state space layer) and `rglru` (Griffin's gated linear recurrent unit); feed-forwards dense with squared
+    relu, or a mixture of experts with sigmoid scores used as they are; a looped span of layers whose later passes add the embedding output."""
+    layers = []
+    for ly in c["layers"]:
+        m = ly["mixer"]
+        if ly["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            qt = a.get("q_temp") or {}
+            left = AttentionMixerConfig(int(a["heads"]), int(a.get("kv_heads", a["heads"])), int(a["dim"]), int(a.get("vdim", a["dim"])), None,
+                                        float(a["scale"]), bias=True, sink_score=0.0, row_norm=True, temp_coef=float(qt.get("coef", 0.0)),
+                                        temp_every=float(qt.get("every", 1.0)))
+            right = StateSpaceMixerConfig(int(r["heads"]), int(r["state"]), int(r["vdim"]), int(r.get("groups", 1)), int(r["conv"]),
+                                          int(r.get("norm_groups", 1)))
+            if left.heads % left.kv_heads or right.heads % right.groups or (right.heads * right.vdim) % right.norm_groups:
+                raise ValueError("kv_heads and groups divide their heads, norm_groups divides heads * vdim")
+            mixer = ParallelMixerConfig(left, right, branch_norm=False, left_scale=float(m.get("left_scale", 1.0)),
+                                        right_scale=float(m.get("right_scale", 1.0)))
+        elif ly["type"] == "rglru":
+            mixer = GatedUnitMixerConfig(int(m["width"]), int(m.get("blocks", 1)), int(m["conv"]))
+            if mixer.width % mixer.blocks:
+                raise ValueError("blocks divide the recurrent width")
+        else:
+            raise ValueError(f"unknown mixer type {ly['type']!r}")
+        mlp = ly.get("mlp")
+        if mlp is None:
+            ff = None
+        elif mlp.get("kind") == "dense":
+            ff = MlpConfig("dense", int(mlp["ff"]), gated=False, act="relu2")
+        elif mlp.get("kind") == "moe":
+            r = mlp["router"]
+            ff = MoeConfig(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), math.inf, alpha=1.0, up_shift=0.0, router="sigmoid",
+                           renormalize=False, weight_scale=float(r.get("scale", 1.0)))
+            if not 1 <= ff.top <= ff.experts:
+                raise ValueError("router: 1 <= top <= experts")
+        else:
+            raise ValueError(f"unknown feed-forward kind {mlp.get('kind')!r}")
+        layers.append(HybridLayerConfig(ly["type"], mixer, ff))
+    lp = c.get("loop") or {}
+    return HybridConfig("Tumitar", int(c["vocab"]), int(c["width"]), float(c["norm"]["eps"]), tuple(layers), int(lp.get("start", 0)),
+                        int(lp.get("stop", 0)), int(lp.get("times", 1)), norm_offset=0.0, block="sequential",
+                        embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)), tied_head=True, loop_add=True)
+
+
 # config.json "architecture" -> parser.  The quantised Llama-family models of MODELS are built by qserve_b200.decode.DecodeRunner.
 ARCHITECTURES: Dict[str, Callable[[dict], HybridConfig]] = {"Rizurax": parse_rizurax, "Toderax": parse_toderax, "Nusuvik": parse_nusuvik,
-                                                                 "Zuzezen": parse_zuzezen, "Nagosun": parse_nagosun}
+                                                                 "Zuzezen": parse_zuzezen, "Nagosun": parse_nagosun, "Tumitar": parse_tumitar}
 
 
 def read_model_config(model_dir: str) -> HybridConfig:

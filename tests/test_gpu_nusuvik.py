@@ -126,7 +126,7 @@ def test_grouped_sigmoid_router_kernel(dev, experts, top, groups, keep, width, T
     hd, wd, cd = h.to(dev), wr.to(dev), corr.to(dev)
     route, idx, wt = torch.zeros(T, experts, device=dev), torch.zeros(T, top, dtype=torch.int32, device=dev), torch.zeros(T, top, device=dev)
     check(lib.qs_hyb_moe_router(route.data_ptr(), idx.data_ptr(), wt.data_ptr(), hd.data_ptr(), wd.data_ptr(), T, width, experts, top, 1, cd.data_ptr(),
-                                groups, keep, 1, _raw()))
+                                groups, keep, 1, 1.0, 1, _raw()))
     spec = {"router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
     want_idx, want_w = O.route(spec, {"router": wr, "correction": corr}, "", h.double())
     assert torch.equal(idx.cpu().long(), want_idx)
