@@ -74,6 +74,9 @@ def parse():
                     "(sandwich blocks with grouped norms and residual gates, windowed attention with capped scores and unit-RMS values, windowed "
                     "latent attention; random weights) at layer sizes of real models, beside the Zuzezen decoder at equal size and its like "
                     "kernels; prints one JSON line")
+    ap.add_argument("--tumitar", action="store_true", help="instead of the default workload: prefill and decode throughput of the Tumitar decoder "
+                    "(attention beside a state space layer, gated linear recurrent units, squared-relu and expert feed-forwards; random weights) at "
+                    "layer sizes of real models, beside the Toderax decoder at equal size and its like kernels; prints one JSON line")
     return ap.parse_args()
 
 
@@ -1461,6 +1464,157 @@ def nagosun_block(args):
 
 
 # ------------------------------------------------------------------------------------------------------------
+# --tumitar: the Tumitar decoder beside the closest existing model (the Toderax decoder on one stream) at equal size
+# ------------------------------------------------------------------------------------------------------------
+def tumitar_block(args):
+    """Prefill and decode (HYBRID_LOAD) of a four-layer Tumitar stack gated unit + dense | attention with state space + experts, twice (32 experts, 8 per
+    token, that hold as many weights per token as the dense feed-forward), beside a Toderax stack on one stream of the same layout (gate
+    recurrence | attention with retention), width, head geometry and experts; then each Tumitar kernel beside the like kernel of Toderax (attention of whole
+    contexts with a sink; retention and gate recurrence for the recurrent layers; the streams' kernel; the router) or of the other designs
+    (gated linear attention; gelu) on the same batches."""
+    import torch
+
+    from qserve_b200._lib import check, lib
+    from qserve_b200.engine import Engine
+    from qserve_b200.hybrid import HybridDecoder, _bmm_f32, random_weights
+    from qserve_b200.modelcfg import (AttentionMixerConfig, GatedLinearMixerConfig, GatedUnitMixerConfig, GateRecurrenceMixerConfig, HybridConfig,
+                                      HybridLayerConfig, MlpConfig, MoeConfig, ParallelMixerConfig, RetentionMixerConfig, RotaryConfig,
+                                      StateSpaceMixerConfig)
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm_gbs = peaks()[0]
+    try:
+        tflops = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"]
+    except (OSError, KeyError, ValueError):
+        tflops = 1590.0
+    stream = torch.cuda.current_stream()
+    reps = max(3, args.kernel_reps)
+    raw = lambda: torch._C._cuda_getCurrentRawStream(0)
+    (B, CTX, NP, LP), E, TOP, N, P, SG = HYBRID_LOAD, 32, 8, 128, 64, 8
+    T = NP * LP
+    out = {"metric": "Tumitar decoder throughput (tokens/s, random weights, bf16, 4 layers)", "unit": "tokens/s", "impl": "ours", "dtype": "bf16",
+           "data": "synthetic", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops}, "load": {"decode_batch": B, "ctx": CTX, "prompts": NP, "prompt": LP},
+           "sizes": {}}
+    pairs = NP * (LP * (LP + 1) // 2)
+
+    def attention_rec(tp, td, H, G, D):
+        return {"prefill_us": tp * 1e6, "prefill_frac_of_measured_bf16_peak": H * pairs * 4 * D / tp / 1e12 / tflops, "decode_us": td * 1e6,
+                "decode_frac_of_measured_hbm": B * (CTX + 1) * G * 2 * D * 2 / td / 1e9 / hbm_gbs}
+
+    def state_rec(tp, td, cells):  # cells: numbers of a sequence's state; an update is a decay, a write and a read: 5 flops
+        return {"prefill_us": tp * 1e6, "prefill_state_gflops": 5 * T * cells / tp / 1e9, "decode_us": td * 1e6,
+                "decode_state_frac_of_measured_hbm": B * cells * 8 / td / 1e9 / hbm_gbs}
+
+    def hbm_rec(t, n_bytes):
+        return {"us": t * 1e6, "frac_of_measured_hbm": n_bytes / t / 1e9 / hbm_gbs}
+
+    for name, (W, H, G, D, FF, V) in HYBRID_SIZES.items():
+        SH = 2 * W // P
+        att = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, sink_score=0.0, row_norm=True, temp_coef=0.1, temp_every=256.0)
+        ssd = StateSpaceMixerConfig(SH, N, P, SG, 4, SG)
+        unit = GatedUnitMixerConfig(W, 16, 4)
+        moe = MoeConfig(E, TOP, FF // TOP, float("inf"), alpha=1.0, up_shift=0.0, router="sigmoid", renormalize=False, weight_scale=2.0)
+        dense = MlpConfig("dense", FF, gated=False, act="relu2")
+        par = ParallelMixerConfig(att, ssd, branch_norm=False, left_scale=0.6, right_scale=0.5)
+        pair = (HybridLayerConfig("rglru", unit, dense), HybridLayerConfig("parallel", par, moe))
+        cfg = HybridConfig("Tumitar", V, W, 1e-5, pair * 2, norm_offset=0.0, block="sequential", embed_scale=8.0, tied_head=True, loop_add=True)
+        tatt = AttentionMixerConfig(H, G, D, D, None, D ** -0.5, bias=True, qk_norm=True, head_temp=True, sink=True, chunk=LP)
+        ret = RetentionMixerConfig(H // 2, D, D, RotaryConfig(D, 1e6, layout="half"), tuple(1.0 - 2.0 ** (-5 - 5 * i / (H // 2)) for i in range(H // 2)))
+        gate = GateRecurrenceMixerConfig(H, D, D)
+        tmoe = MoeConfig(E, TOP, FF // TOP, 7.0, FF // TOP, 7.0)
+        tcfg = HybridConfig("Toderax", V, W, 1e-5, (HybridLayerConfig("hgrn2", gate, tmoe), HybridLayerConfig("parallel", ParallelMixerConfig(tatt, ret), tmoe)) * 2,
+                            norm_offset=0.0, block="sequential", streams=1, norm_groups=8, embed_scale=4.0)
+        g = torch.Generator().manual_seed(0)
+        kern, like = {}, {}
+        with torch.no_grad():
+            model = HybridDecoder(cfg, random_weights(cfg, 0, dev), torch.bfloat16, dev)
+            eng = Engine(model, max_tokens=B * (CTX + 64) + NP * LP, max_seqs=B + NP)
+            rec, pb, db = hybrid_steps(model, eng, V, g, reps, stream)
+
+            def lone_times(m):
+                mixer = hybrid_lone_mixer(m, W, 1, dev)
+                return hybrid_mixer_times(mixer, eng.cache.mixer_storage(m), pb, db, T, reps, stream)
+
+            kern["attention(bias+row norms+temperature+append, tiles / head groups with a spare term)"] = attention_rec(*lone_times(att), H, G, D)
+            like["attention(bias+unit RMS+append, tiles / head groups with a sink)"] = attention_rec(*lone_times(tatt), H, G, D)
+            kern["state_space(convolution+step sizes, scan, gate+part norm)"] = state_rec(*lone_times(ssd), SH * N * P)
+            like["retention(rotate, scan, unit RMS+gate)"] = state_rec(*lone_times(ret), H // 2 * D * D)
+            like["gate_recurrence(prepare, scan, unit RMS)"] = state_rec(*lone_times(gate), H * D * D)
+            like["gated_linear(decay product+prepare, scan, unit RMS+gate)"] = state_rec(*lone_times(GatedLinearMixerConfig(H, D, D, 8.0, 32)), H * D * D)
+            tp, td = lone_times(unit)
+            # the gate product's flops beside the bytes: projections in, u out and in again, fp32 logits out and in, output
+            kern["gated_unit(convolution, gate product, tile scans+gelu branch)"] = {
+                "prefill": hbm_rec(tp, T * W * (4 + 2 + 2 + 8 + 8 + 2 + 2)), "decode_us": td * 1e6}
+            mixer = hybrid_lone_mixer(unit, W, 1, dev)
+            store = eng.cache.mixer_storage(unit)
+            proj, u = torch.randn(T, 2 * W, device=dev).to(torch.bfloat16), torch.empty(T, W, dtype=torch.bfloat16, device=dev)
+            p = lambda t: t.data_ptr()
+            tables = lambda b: (p(b.entry_start), p(b.entry_len), p(b.entry_slot), p(b.entry_pos0))
+            tc = time_kernel(lambda: (check(lib.qs_hyb_lru_conv(p(u), p(proj), 2 * W, p(mixer.x_bias), p(mixer.conv_w), p(mixer.conv_b), p(store["conv"]), p(pb.tok_entry),
+                                                                p(pb.tok_pos), *tables(pb), T, NP, W, 4, 0, raw())), 1)[1], reps, stream)
+            kern["gated_unit: convolution"] = hbm_rec(tc, T * W * 4)
+            tz = time_kernel(lambda: (_bmm_f32(u.view(T, unit.blocks, -1).transpose(0, 1), mixer.w_gates.transpose(1, 2)), 1)[1], reps, stream)
+            kern["gated_unit: gate product (library)"] = hbm_rec(tz, T * W * 10)
+            z = torch.randn(unit.blocks, T, 2 * W // unit.blocks, device=dev)
+            h1, sums = torch.empty(T, W, dtype=torch.bfloat16, device=dev), torch.empty(mixer.scratch_floats(T), device=dev)
+            scan = lambda b, n: check(lib.qs_hyb_lru_scan(p(h1), W, p(store["state"]), p(sums), p(u), p(z), p(proj), 2 * W, p(mixer.y_bias), p(mixer.r_bias), p(mixer.i_bias),
+                                                          p(mixer.rate), p(b.tile_entry), p(b.tile_row0), b.n_tiles, b.n_short, *tables(b), n, b.n_entries, W,
+                                                          unit.blocks, 64, 16, 0, raw()))
+            ts = time_kernel(lambda: (scan(pb, T), 1)[1], reps, stream)
+            kern["gated_unit: tile scans+gelu branch"] = hbm_rec(ts, T * W * 14)   # logits 8, u 2, y 2, output 2 (once)
+            ts = time_kernel(lambda: (scan(db, B), 1)[1], reps * 4, stream)
+            kern["gated_unit: scan, decode batch"] = {"us": ts * 1e6}
+            del mixer, store, proj, u, z, sums
+            x, y, w1 = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev), torch.ones(W, device=dev)
+            upd = torch.zeros(T, W, dtype=torch.bfloat16, device=dev)
+            for label, n, r_ in (("prefill", T, reps), ("decode batch", B, reps * 4)):
+                tn = time_kernel(lambda: (check(lib.qs_hyb_stream_update_norm(p(h1), None, p(x), None, p(y), 1, None, 0, None, p(w1), None, 1, 1e-5, n, W, 0, raw())), 1)[1],
+                                 r_, stream)
+                kern[f"stream_update_norm(fp32 rows in, residual, norm), {label}"] = hbm_rec(tn, n * W * 14)
+                tn = time_kernel(lambda: (check(lib.qs_hyb_stream_norm(p(h1), None, p(x), 1, p(upd), 0, p(w1), p(w1), p(w1), p(w1), 8, 0.0, 1e-5, n, W, 0, raw())), 1)[1], r_,
+                                 stream)
+                like[f"stream_norm(bf16 rows in, one stream, group norm), {label}"] = hbm_rec(tn, n * W * 12)
+            a, gu, up = torch.empty(T, FF, dtype=torch.bfloat16, device=dev), torch.randn(T, 2 * FF, device=dev).to(torch.bfloat16), torch.randn(T, FF, device=dev).to(torch.bfloat16)
+            tg = time_kernel(lambda: (check(lib.qs_hyb_bias_relu_squared(p(a), FF, p(up), FF, None, T, FF, 0, raw())), 1)[1], reps, stream)
+            kern["relu_squared"] = hbm_rec(tg, T * FF * 4)
+            tg = time_kernel(lambda: (check(lib.qs_hyb_bias_gelu_tanh(p(a), FF, p(up), FF, None, T, FF, 0, raw())), 1)[1], reps, stream)
+            like["gelu_tanh"] = hbm_rec(tg, T * FF * 4)
+            del a, gu, up, y, upd
+            h = torch.randn(T, W, device=dev).to(torch.bfloat16)
+            ff = model.layers[1].ff
+            route, ti, tw = torch.empty(T, E, device=dev), torch.empty(T, TOP, dtype=torch.int32, device=dev), torch.empty(T, TOP, device=dev)
+            for label, table, mode, renorm in (("sigmoid, weights as they are", kern, 1, 0), ("softmax", like, 0, 1)):
+                tr = time_kernel(lambda: (check(lib.qs_hyb_moe_router(p(route), p(ti), p(tw), p(h), p(ff.w_router), T, W, E, TOP, mode, None, 1, 1, renorm, 2.0, 0, raw())), 1)[1],
+                                 reps, stream)
+                table[f"moe_router({label})"] = hbm_rec(tr, T * W * 2)
+            for label, hh, r_ in (("prefill", h, reps), ("decode", h[:B].contiguous(), reps * 4)):
+                n = hh.shape[0]
+                tm = time_kernel(lambda: (ff.run(hh, 0, raw()), 1)[1], r_, stream)
+                kern[f"moe_feed_forward_{label}(router+sort+gather+2 grouped products+act+combine)"] = {
+                    "us": tm * 1e6, "frac_of_measured_bf16_peak": n * 6 * W * TOP * moe.ff / tm / 1e12 / tflops,
+                    "weights_frac_of_measured_hbm": 3 * W * min(E, n * TOP) * moe.ff * 2 / tm / 1e9 / hbm_gbs}
+            del eng, model, x, h1, h, ff
+            torch.cuda.empty_cache()
+            model = HybridDecoder(tcfg, random_weights(tcfg, 0, dev), torch.bfloat16, dev)
+            eng = Engine(model, max_tokens=B * (CTX + 64) + NP * LP, max_seqs=B + NP)
+            peer, _, _ = hybrid_steps(model, eng, V, g, reps, stream)
+            ff = model.layers[1].ff
+            h = torch.randn(T, W, device=dev).to(torch.bfloat16)
+            for label, hh, r_ in (("prefill", h, reps), ("decode", h[:B].contiguous(), reps * 4)):
+                n = hh.shape[0]
+                tm = time_kernel(lambda: (ff.run(hh, 0, raw()), 1)[1], r_, stream)
+                like[f"moe_feed_forward_{label}(the same and a shared expert)"] = {
+                    "us": tm * 1e6, "frac_of_measured_bf16_peak": n * 6 * W * (TOP * tmoe.ff + tmoe.shared_ff) / tm / 1e12 / tflops,
+                    "weights_frac_of_measured_hbm": 3 * W * (min(E, n * TOP) * tmoe.ff + tmoe.shared_ff) * 2 / tm / 1e9 / hbm_gbs}
+            del eng, model, h, ff
+        torch.cuda.empty_cache()
+        rec["kernels"], rec["like_kernels"], rec["toderax_equal_size"] = kern, like, peer
+        out["sizes"][name] = rec
+    print(json.dumps(out), flush=True)
+
+
+# ------------------------------------------------------------------------------------------------------------
 def main():
     args = parse()
     rank = int(os.environ.get("RANK", "0"))
@@ -1488,6 +1642,10 @@ def main():
     if args.nagosun:
         if rank == 0:
             nagosun_block(args)
+        return
+    if args.tumitar:
+        if rank == 0:
+            tumitar_block(args)
         return
     if args.impl == "reference-gpu":
         if rank == 0:
