@@ -73,6 +73,75 @@ __device__ __forceinline__ void conv_row(float (&y)[V], const ST* __restrict__ i
   }
 }
 
+// The same for a walk over neighbouring rows, `TAPS` known: the channels' weights and the window of inputs stay in registers.
+template <typename ST, int V, int TAPS>
+struct ConvWalk {
+  float w[V][TAPS], b[V], xb[V], x[TAPS][V];
+  int entry = -1;
+
+  __device__ __forceinline__ ConvWalk(const float* __restrict__ cw, const float* __restrict__ cb, const float* __restrict__ in_bias, int c) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      b[v] = cb != nullptr ? cb[c + v] : 0.f;
+      xb[v] = in_bias != nullptr ? in_bias[c + v] : 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[v][j] = cw[(size_t)(c + v) * TAPS + j];
+    }
+  }
+  __device__ __forceinline__ void row(float (&y)[V], const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias, float* st, int t, int e,
+                                      int local, int pos, int C, int c, bool shift) {
+    if (e != entry) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) conv_input<ST, V>(x[j], in, stride, in_bias, st, t, local, pos, TAPS - 1 - j, TAPS, C, c);
+      entry = e;
+    } else {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int v = 0; v < V; ++v) x[j][v] = x[j + 1][v];
+    }
+    const ST* p = in + (size_t)t * stride + c;
+    if constexpr (V == 4) {
+      const float4 q = ld4(p);
+      x[TAPS - 1][0] = q.x; x[TAPS - 1][1] = q.y; x[TAPS - 1][2] = q.z; x[TAPS - 1][3] = q.w;
+    } else {
+      x[TAPS - 1][0] = ldf(p);
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      x[TAPS - 1][v] += xb[v];
+      y[v] = b[v];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) y[v] += w[v][j] * x[j][v];
+    }
+    if (shift) {
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j)
+#pragma unroll
+        for (int v = 0; v < V; ++v) st[(size_t)(j - 1) * C + c + v] = x[j][v];
+    }
+  }
+};
+// any number of taps
+template <typename ST, int V>
+struct ConvWalk<ST, V, 0> {
+  const float *cw, *cb;
+  int taps;
+  __device__ __forceinline__ ConvWalk(const float* w, const float* b, int n) : cw(w), cb(b), taps(n) {}
+  __device__ __forceinline__ void row(float (&y)[V], const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias, float* st, int t, int,
+                                      int local, int pos, int C, int c, bool shift) {
+    conv_row<ST, V>(y, in, stride, in_bias, st, cw, cb, t, local, pos, taps, C, c, shift);
+  }
+};
+template <typename ST, int V, int TAPS>
+__device__ __forceinline__ ConvWalk<ST, V, TAPS> conv_walk(const float* w, const float* b, const float* in_bias, int taps, int c) {
+  if constexpr (TAPS == 0) return ConvWalk<ST, V, 0>(w, b, taps);
+  else return ConvWalk<ST, V, TAPS>(w, b, in_bias, c);
+}
+
+// silu as the storage type needs it: the special-function unit's exponential and division for bfloat16 results, the exact ones for fp32
+template <typename ST> __device__ __forceinline__ float silu_as(float z) { return sizeof(ST) == 2 ? z * fast_sigmoid(z) : silu_f(z); }
+
 // the sequence's convolution state after a portion: its last taps - 1 inputs (older ones shift out)
 template <typename ST>
 __global__ void conv_state_kernel(float* __restrict__ conv_state, const ST* __restrict__ in, long long stride, const float* __restrict__ in_bias,
@@ -100,7 +169,7 @@ __global__ void conv_state_kernel(float* __restrict__ conv_state, const ST* __re
 //   a = exp(-exp(A_log) dt)
 // grid (runs of `run` tokens, blocks of 128 V channels)
 // ---------------------------------------------------------------------------------------------------------------------------------
-template <typename ST, int V>
+template <typename ST, int V, int TAPS>
 __global__ void __launch_bounds__(128) ssd_prepare_kernel(float* __restrict__ prep, const ST* __restrict__ proj, long long stride,
                                                           const float* __restrict__ conv_w, const float* __restrict__ conv_b, float* conv_state,
                                                           const float* __restrict__ a_log, const float* __restrict__ dt_bias,
@@ -110,15 +179,15 @@ __global__ void __launch_bounds__(128) ssd_prepare_kernel(float* __restrict__ pr
   const int inner = H * Dv, C = inner + 2 * G * N, P = ssd_row_floats(H, G, N, Dv);
   const int c = (blockIdx.y * 128 + threadIdx.x) * V;
   const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+  auto walk = conv_walk<ST, V, TAPS>(conv_w, conv_b, nullptr, taps, min(c, C - V));
   for (int t = t0; t < t1; ++t) {
     const int e = tok_entry[t];
     float* o = prep + (size_t)t * P;
     if (c < C) {
       float y[V];
-      conv_row<ST, V>(y, proj + inner, stride, nullptr, conv_state + (size_t)entry_slot[e] * (taps - 1) * C, conv_w, conv_b, t, t - entry_start[e],
-                      tok_pos[t], taps, C, c, shift != 0);
+      walk.row(y, proj + inner, stride, nullptr, conv_state + (size_t)entry_slot[e] * (taps - 1) * C, t, e, t - entry_start[e], tok_pos[t], C, c, shift != 0);
 #pragma unroll
-      for (int v = 0; v < V; ++v) y[v] = silu_f(y[v]);
+      for (int v = 0; v < V; ++v) y[v] = silu_as<ST>(y[v]);
       if constexpr (V == 4) st4(o + c, make_float4(y[0], y[1], y[2], y[3]));
       else o[c] = y[0];
     }
@@ -149,13 +218,13 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(ST* __restrict__ out, long
     for (int i = threadIdx.x * 4; i < part; i += blockDim.x * 4) {
       float4 a = ld4(yr + i);
       const float4 g = ld4(zr + i);
-      a.x *= silu_f(g.x); a.y *= silu_f(g.y); a.z *= silu_f(g.z); a.w *= silu_f(g.w);
+      a.x *= silu_as<ST>(g.x); a.y *= silu_as<ST>(g.y); a.z *= silu_as<ST>(g.z); a.w *= silu_as<ST>(g.w);
       ss += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
       st4(ys + i, a);
     }
   } else {
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
-      const float a = yr[i] * silu_f(ldf(zr + i));
+      const float a = yr[i] * silu_as<ST>(ldf(zr + i));
       ss += a * a;
       ys[i] = a;
     }
@@ -175,7 +244,7 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(ST* __restrict__ out, long
 // gated linear unit.  projection row: [W y | W x] (biases not yet added)
 // step 1: u = convolution of x + x_bias, in the storage type [T][W]
 // ---------------------------------------------------------------------------------------------------------------------------------
-template <typename ST, int V>
+template <typename ST, int V, int TAPS>
 __global__ void __launch_bounds__(128) lru_conv_kernel(ST* __restrict__ u, const ST* __restrict__ proj, long long stride, const float* __restrict__ x_bias,
                                                        const float* __restrict__ conv_w, const float* __restrict__ conv_b, float* conv_state,
                                                        const int* __restrict__ tok_entry, const int* __restrict__ tok_pos,
@@ -184,11 +253,11 @@ __global__ void __launch_bounds__(128) lru_conv_kernel(ST* __restrict__ u, const
   const int c = (blockIdx.y * 128 + threadIdx.x) * V;
   if (c >= W) return;
   const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+  auto walk = conv_walk<ST, V, TAPS>(conv_w, conv_b, x_bias, taps, c);
   for (int t = t0; t < t1; ++t) {
     const int e = tok_entry[t];
     float y[V];
-    conv_row<ST, V>(y, proj + W, stride, x_bias, conv_state + (size_t)entry_slot[e] * (taps - 1) * W, conv_w, conv_b, t, t - entry_start[e], tok_pos[t],
-                    taps, W, c, shift != 0);
+    walk.row(y, proj + W, stride, x_bias, conv_state + (size_t)entry_slot[e] * (taps - 1) * W, t, e, t - entry_start[e], tok_pos[t], W, c, shift != 0);
     if constexpr (V == 4) st4(u + (size_t)t * W + c, make_float4(y[0], y[1], y[2], y[3]));
     else stf(u + (size_t)t * W + c, y[0]);
   }
@@ -214,7 +283,20 @@ __device__ __forceinline__ LruChannel lru_channel(const float* z, const float* r
   k.rate = rate[c];
   return k;
 }
+// FAST (bfloat16 storage): fp32 throughout, with the special-function unit's exponentials, divisions and square root (relative error about 2^-21) and
+// 1 - a^2 = -expm1(x), x = 2 log a, from the exponential series where a^2 is close to 1
+template <bool FAST>
 __device__ __forceinline__ void lru_gates(float& a, float& b, float zr, float zi, float u, const LruChannel& k) {
+  if (FAST) {
+    const float la = k.rate * fast_sigmoid(zr + k.rb), x = 2.f * la;
+    a = fast_exp2(la * 1.4426950408889634f);
+    const float series = -x * (1.f + x * (1.f / 2.f) * (1.f + x * (1.f / 3.f) * (1.f + x * (1.f / 4.f) * (1.f + x * (1.f / 5.f) * (1.f + x * (1.f / 6.f))))));
+    const float m = x > -0.25f ? series : 1.f - a * a;
+    float root;
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(m));
+    b = root * fast_sigmoid(zi + k.ib) * u;
+    return;
+  }
   const float la = k.rate * sigmoid_f(zr + k.rb);
   a = expf(la);
   b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + k.ib) * u;
@@ -247,7 +329,7 @@ __global__ void __launch_bounds__(128) lru_tile_sums_kernel(float* __restrict__ 
     for (int q = 0; q < kLruBatch; ++q) {
       if (j + q >= n) break;
       float a, b;
-      lru_gates(a, b, zr[q], zi[q], uu[q], k);
+      lru_gates<sizeof(ST) == 2>(a, b, zr[q], zi[q], uu[q], k);
       A *= a;
       S = a * S + b;
     }
@@ -308,10 +390,11 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(ST* __restrict__ out, lon
     for (int q = 0; q < kLruBatch; ++q) {
       if (j + q >= n) break;
       float a, b;
-      lru_gates(a, b, zr[q], zi[q], uu[q], k);
+      lru_gates<sizeof(ST) == 2>(a, b, zr[q], zi[q], uu[q], k);
       S = a * S + b;
-      const float g = yy[q] + yb;  // gelu_tanh(g) = g / (1 + e^(-2 sqrt(2/pi) (g + 0.044715 g^3)))
-      stf(out + (size_t)(s0 + j + q) * out_stride + c, S * (g / (1.f + expf(-2.f * 0.7978845608028654f * (g + 0.044715f * g * g * g)))));
+      const float g = yy[q] + yb, v = 2.f * 0.7978845608028654f * (g + 0.044715f * g * g * g);
+      const float gelu = g * (sizeof(ST) == 2 ? fast_sigmoid(v) : sigmoid_f(v));   // 0.5 (1 + tanh(v / 2)) = sigmoid(v)
+      stf(out + (size_t)(s0 + j + q) * out_stride + c, S * gelu);
     }
   }
   if (r0 + n == len) *slot = S;
@@ -328,7 +411,7 @@ int launch_conv_state(float* conv_state, const ST* in, long long stride, const f
 bool aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
 
 // tokens a block of a convolution kernel walks: neighbours find each other's rows in the cache once there are blocks enough
-int conv_run(int T) { return T >= 2048 ? 8 : T >= 512 ? 4 : 1; }
+int conv_run(int T) { return T >= 2048 ? 16 : T >= 512 ? 4 : 1; }
 
 template <typename ST>
 int launch_state_space(void* out, long long out_stride, float* prep, float* o_raw, const void* proj_, long long stride, const float* conv_w,
@@ -340,7 +423,8 @@ int launch_state_space(void* out, long long out_stride, float* prep, float* o_ra
   const int inner = H * Dv, C = inner + 2 * G * N, run = conv_run(T), shift = T == E && taps > 1;
   const bool v4 = C % 4 == 0 && inner % 4 == 0 && stride % 4 == 0 && aligned(proj, 4 * sizeof(ST)) && aligned(prep, 16);
   dim3 grid((T + run - 1) / run, (C + (v4 ? 512 : 128) - 1) / (v4 ? 512 : 128));
-  auto prepare = v4 ? ssd_prepare_kernel<ST, 4> : ssd_prepare_kernel<ST, 1>;
+  auto prepare = !v4 ? ssd_prepare_kernel<ST, 1, 0> : taps == 4 ? ssd_prepare_kernel<ST, 4, 4> : taps == 3 ? ssd_prepare_kernel<ST, 4, 3>
+                 : taps == 2 ? ssd_prepare_kernel<ST, 4, 2> : ssd_prepare_kernel<ST, 4, 0>;
   prepare<<<grid, 128, 0, s>>>(prep, proj, stride, conv_w, conv_b, conv_state, a_log, dt_bias, tok_entry, tok_pos, entry_start, entry_slot, T, H, G, N, Dv,
                                taps, run, shift);
   if (!shift)
@@ -363,7 +447,8 @@ int launch_lru_conv(void* u, const void* proj_, long long stride, const float* x
   const int run = conv_run(T), shift = T == E && taps > 1;
   const bool v4 = W % 4 == 0 && stride % 4 == 0 && aligned(proj, 4 * sizeof(ST)) && aligned(u, 4 * sizeof(ST));
   dim3 grid((T + run - 1) / run, (W + (v4 ? 512 : 128) - 1) / (v4 ? 512 : 128));
-  auto conv = v4 ? lru_conv_kernel<ST, 4> : lru_conv_kernel<ST, 1>;
+  auto conv = !v4 ? lru_conv_kernel<ST, 1, 0> : taps == 4 ? lru_conv_kernel<ST, 4, 4> : taps == 3 ? lru_conv_kernel<ST, 4, 3>
+              : taps == 2 ? lru_conv_kernel<ST, 4, 2> : lru_conv_kernel<ST, 4, 0>;
   conv<<<grid, 128, 0, s>>>((ST*)u, proj, stride, x_bias, conv_w, conv_b, conv_state, tok_entry, tok_pos, entry_start, entry_slot, T, W, taps, run, shift);
   if (!shift) return launch_conv_state<ST>(conv_state, proj + W, stride, x_bias, entry_start, entry_len, entry_slot, entry_pos0, E, W, taps, s);
   return check_cuda(cudaGetLastError(), "hyb_lru_conv");
