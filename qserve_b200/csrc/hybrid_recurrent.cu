@@ -266,99 +266,141 @@ __global__ void __launch_bounds__(128) lru_conv_kernel(ST* __restrict__ u, const
 // step 2 (between the kernels): gate logits z fp32 [blocks][T][2 W / blocks]: a block's r logits, then its i logits.
 // step 3: the recurrence.  One token of one channel: r = sigmoid(z_r + r_bias), i = sigmoid(z_i + i_bias), log a = rate * r (rate < 0 per
 // channel), S <- a S + sqrt(1 - a^2) i u with 1 - a^2 = -expm1(2 log a).
-struct LruChannel {
-  const float* zr;    // r logit of row 0; rows are zs floats apart
-  size_t zs, zi;      // zi: distance of the i logit
-  float rb, ib, rate;
+// A thread owns V neighbouring channels of one block (V = 2: the channels of a block are even in number and aligned).
+template <int V>
+struct LruChannels {
+  const float* zr;    // r logits of row 0; rows are zs floats apart
+  size_t zs, zi;      // zi: distance of the i logits
+  float rb[V], ib[V], rate[V];
+
+  __device__ __forceinline__ LruChannels(const float* z, const float* r_bias, const float* i_bias, const float* rates, int T, int W, int blocks, int c) {
+    const int wb = W / blocks, b = c / wb, j = c - b * wb;
+    zr = z + (size_t)b * T * 2 * wb + j;
+    zs = 2 * (size_t)wb;
+    zi = wb;
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      rb[v] = r_bias[c + v];
+      ib[v] = i_bias[c + v];
+      rate[v] = rates[c + v];
+    }
+  }
 };
-__device__ __forceinline__ LruChannel lru_channel(const float* z, const float* r_bias, const float* i_bias, const float* rate, int T, int W, int blocks,
-                                                  int c) {
-  const int wb = W / blocks, b = c / wb, j = c - b * wb;
-  LruChannel k;
-  k.zr = z + (size_t)b * T * 2 * wb + j;
-  k.zs = 2 * (size_t)wb;
-  k.zi = wb;
-  k.rb = r_bias[c];
-  k.ib = i_bias[c];
-  k.rate = rate[c];
-  return k;
+template <int V> __device__ __forceinline__ void load_row(float (&x)[V], const float* p) {
+  if constexpr (V == 2) {
+    const float2 q = *reinterpret_cast<const float2*>(p);
+    x[0] = q.x; x[1] = q.y;
+  } else {
+    x[0] = *p;
+  }
 }
+template <int V> __device__ __forceinline__ void load_row(float (&x)[V], const __nv_bfloat16* p) {
+  if constexpr (V == 2) {
+    const uint32_t q = *reinterpret_cast<const uint32_t*>(p);
+    x[0] = __uint_as_float(q << 16); x[1] = __uint_as_float(q & 0xffff0000u);
+  } else {
+    x[0] = ldf(p);
+  }
+}
+template <int V> __device__ __forceinline__ void store_row(float* p, const float (&x)[V]) {
+#pragma unroll
+  for (int v = 0; v < V; ++v) p[v] = x[v];
+}
+template <int V> __device__ __forceinline__ void store_row(__nv_bfloat16* p, const float (&x)[V]) {
+  if constexpr (V == 2) *reinterpret_cast<uint32_t*>(p) = pack_bf16(x[0], x[1]);
+  else stf(p, x[0]);
+}
+
 // FAST (bfloat16 storage): fp32 throughout, with the special-function unit's exponentials, divisions and square root (relative error about 2^-21) and
 // 1 - a^2 = -expm1(x), x = 2 log a, from the exponential series where a^2 is close to 1
 template <bool FAST>
-__device__ __forceinline__ void lru_gates(float& a, float& b, float zr, float zi, float u, const LruChannel& k) {
+__device__ __forceinline__ void lru_gates(float& a, float& b, float zr, float zi, float u, float rate) {
   if (FAST) {
-    const float la = k.rate * fast_sigmoid(zr + k.rb), x = 2.f * la;
+    const float la = rate * fast_sigmoid(zr), x = 2.f * la;
     a = fast_exp2(la * 1.4426950408889634f);
     const float series = -x * (1.f + x * (1.f / 2.f) * (1.f + x * (1.f / 3.f) * (1.f + x * (1.f / 4.f) * (1.f + x * (1.f / 5.f) * (1.f + x * (1.f / 6.f))))));
     const float m = x > -0.25f ? series : 1.f - a * a;
     float root;
     asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(m));
-    b = root * fast_sigmoid(zi + k.ib) * u;
+    b = root * fast_sigmoid(zi) * u;
     return;
   }
-  const float la = k.rate * sigmoid_f(zr + k.rb);
+  const float la = rate * sigmoid_f(zr);
   a = expf(la);
-  b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + k.ib) * u;
+  b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi) * u;
 }
 
 constexpr int kLruBatch = 4;  // tokens whose inputs are on their way at once
 
 // what a tile of rows does to a state: S <- A S + B.  sums [n_tiles][2][W]
-template <typename ST>
+template <typename ST, int V>
 __global__ void __launch_bounds__(128) lru_tile_sums_kernel(float* __restrict__ sums, const ST* __restrict__ u, const float* __restrict__ z,
                                                             const float* __restrict__ r_bias, const float* __restrict__ i_bias,
                                                             const float* __restrict__ rate, const int* __restrict__ tile_entry,
                                                             const int* __restrict__ tile_row0, const int* __restrict__ entry_start,
                                                             const int* __restrict__ entry_len, int T, int W, int blocks, int tile_rows) {
-  const int c = blockIdx.y * 128 + threadIdx.x, tile = blockIdx.x;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * V, tile = blockIdx.x;
   if (c >= W) return;
   const int e = tile_entry[tile], r0 = tile_row0[tile], n = min(tile_rows, entry_len[e] - r0), s0 = entry_start[e] + r0;
-  const LruChannel k = lru_channel(z, r_bias, i_bias, rate, T, W, blocks, c);
-  float A = 1.f, S = 0.f;
+  const LruChannels<V> k(z, r_bias, i_bias, rate, T, W, blocks, c);
+  float A[V], S[V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) { A[v] = 1.f; S[v] = 0.f; }
   for (int j = 0; j < n; j += kLruBatch) {
-    float zr[kLruBatch], zi[kLruBatch], uu[kLruBatch];
+    float zr[kLruBatch][V], zi[kLruBatch][V], uu[kLruBatch][V];
 #pragma unroll
     for (int q = 0; q < kLruBatch; ++q) {
       const size_t t = s0 + min(j + q, n - 1);
-      zr[q] = k.zr[t * k.zs];
-      zi[q] = k.zr[t * k.zs + k.zi];
-      uu[q] = ldf(u + t * W + c);
+      load_row<V>(zr[q], k.zr + t * k.zs);
+      load_row<V>(zi[q], k.zr + t * k.zs + k.zi);
+      load_row<V>(uu[q], u + t * W + c);
     }
 #pragma unroll
     for (int q = 0; q < kLruBatch; ++q) {
       if (j + q >= n) break;
-      float a, b;
-      lru_gates<sizeof(ST) == 2>(a, b, zr[q], zi[q], uu[q], k);
-      A *= a;
-      S = a * S + b;
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        float a, b;
+        lru_gates<sizeof(ST) == 2>(a, b, zr[q][v] + k.rb[v], zi[q][v] + k.ib[v], uu[q][v], k.rate[v]);
+        A[v] *= a;
+        S[v] = a * S[v] + b;
+      }
     }
   }
-  sums[(size_t)tile * 2 * W + c] = A;
-  sums[((size_t)tile * 2 + 1) * W + c] = S;
+  store_row<V>(sums + (size_t)tile * 2 * W + c, A);
+  store_row<V>(sums + ((size_t)tile * 2 + 1) * W + c, S);
 }
 
-// start state of every tile, over the tile's A.  An entry's tiles are neighbours; the block of its first tile walks them.
+// start state of every tile, over the tile's A.  An entry's tiles are neighbours; the block of its first tile walks them, eight at a time.
 __global__ void __launch_bounds__(128) lru_tile_starts_kernel(float* __restrict__ sums, const float* __restrict__ state, const int* __restrict__ tile_entry,
-                                                              const int* __restrict__ tile_row0, const int* __restrict__ entry_slot,
-                                                              const int* __restrict__ entry_pos0, int n_tiles, int W) {
+                                                              const int* __restrict__ tile_row0, const int* __restrict__ entry_len,
+                                                              const int* __restrict__ entry_slot, const int* __restrict__ entry_pos0, int W, int tile_rows) {
+  constexpr int U = 8;
   const int c = blockIdx.y * 128 + threadIdx.x;
-  int tile = blockIdx.x;
-  if (tile_row0[tile] != 0 || c >= W) return;
-  const int e = tile_entry[tile];
+  if (tile_row0[blockIdx.x] != 0 || c >= W) return;
+  const int e = tile_entry[blockIdx.x], n = (entry_len[e] + tile_rows - 1) / tile_rows;
   float S = entry_pos0[e] == 0 ? 0.f : state[(size_t)entry_slot[e] * W + c];
-  do {
-    float* p = sums + (size_t)tile * 2 * W + c;
-    const float A = p[0], B = p[W];
-    p[0] = S;
-    S = A * S + B;
-    ++tile;
-  } while (tile < n_tiles && tile_entry[tile] == e);
+  float* p = sums + (size_t)blockIdx.x * 2 * W + c;
+  for (int i = 0; i < n; i += U) {
+    float A[U], B[U];
+#pragma unroll
+    for (int q = 0; q < U; ++q) {
+      const size_t at = (size_t)min(i + q, n - 1) * 2 * W;
+      A[q] = p[at];
+      B[q] = p[at + W];
+    }
+#pragma unroll
+    for (int q = 0; q < U; ++q) {
+      if (i + q >= n) break;
+      p[(size_t)(i + q) * 2 * W] = S;
+      S = A[q] * S + B[q];
+    }
+  }
 }
 
 // The recurrence over a tile (tiles != 0: start state from sums) or over a whole entry of fewer than long_min tokens (tiles == 0: start state
 // from the slot; longer entries are left to the tiles), read out through the gelu branch.  The slot takes the state after the entry's last row.
-template <typename ST>
+template <typename ST, int V>
 __global__ void __launch_bounds__(128) lru_scan_kernel(ST* __restrict__ out, long long out_stride, float* state, const float* __restrict__ sums,
                                                        const ST* __restrict__ u, const float* __restrict__ z, const ST* __restrict__ y, long long y_stride,
                                                        const float* __restrict__ y_bias, const float* __restrict__ r_bias,
@@ -367,37 +409,45 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(ST* __restrict__ out, lon
                                                        const int* __restrict__ entry_start, const int* __restrict__ entry_len,
                                                        const int* __restrict__ entry_slot, const int* __restrict__ entry_pos0, int tiles, int long_min, int T,
                                                        int W, int blocks, int tile_rows) {
-  const int c = blockIdx.y * 128 + threadIdx.x;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * V;
   const int e = tiles ? tile_entry[blockIdx.x] : blockIdx.x;
   const int len = entry_len[e], r0 = tiles ? tile_row0[blockIdx.x] : 0, n = tiles ? min(tile_rows, len - r0) : len;
   if (c >= W || (!tiles && len >= long_min)) return;
   const int s0 = entry_start[e] + r0;
   float* slot = state + (size_t)entry_slot[e] * W + c;
-  const LruChannel k = lru_channel(z, r_bias, i_bias, rate, T, W, blocks, c);
-  const float yb = y_bias[c];
-  float S = tiles ? sums[(size_t)blockIdx.x * 2 * W + c] : (entry_pos0[e] == 0 ? 0.f : *slot);
+  const LruChannels<V> k(z, r_bias, i_bias, rate, T, W, blocks, c);
+  float yb[V], S[V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    yb[v] = y_bias[c + v];
+    S[v] = tiles ? sums[(size_t)blockIdx.x * 2 * W + c + v] : (entry_pos0[e] == 0 ? 0.f : slot[v]);
+  }
   for (int j = 0; j < n; j += kLruBatch) {
-    float zr[kLruBatch], zi[kLruBatch], uu[kLruBatch], yy[kLruBatch];
+    float zr[kLruBatch][V], zi[kLruBatch][V], uu[kLruBatch][V], yy[kLruBatch][V];
 #pragma unroll
     for (int q = 0; q < kLruBatch; ++q) {
       const size_t t = s0 + min(j + q, n - 1);
-      zr[q] = k.zr[t * k.zs];
-      zi[q] = k.zr[t * k.zs + k.zi];
-      uu[q] = ldf(u + t * W + c);
-      yy[q] = ldf(y + t * y_stride + c);
+      load_row<V>(zr[q], k.zr + t * k.zs);
+      load_row<V>(zi[q], k.zr + t * k.zs + k.zi);
+      load_row<V>(uu[q], u + t * W + c);
+      load_row<V>(yy[q], y + t * y_stride + c);
     }
 #pragma unroll
     for (int q = 0; q < kLruBatch; ++q) {
       if (j + q >= n) break;
-      float a, b;
-      lru_gates<sizeof(ST) == 2>(a, b, zr[q], zi[q], uu[q], k);
-      S = a * S + b;
-      const float g = yy[q] + yb, v = 2.f * 0.7978845608028654f * (g + 0.044715f * g * g * g);
-      const float gelu = g * (sizeof(ST) == 2 ? fast_sigmoid(v) : sigmoid_f(v));   // 0.5 (1 + tanh(v / 2)) = sigmoid(v)
-      stf(out + (size_t)(s0 + j + q) * out_stride + c, S * gelu);
+      float o[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        float a, b;
+        lru_gates<sizeof(ST) == 2>(a, b, zr[q][v] + k.rb[v], zi[q][v] + k.ib[v], uu[q][v], k.rate[v]);
+        S[v] = a * S[v] + b;
+        const float g = yy[q][v] + yb[v], w = 2.f * 0.7978845608028654f * (g + 0.044715f * g * g * g);
+        o[v] = S[v] * g * (sizeof(ST) == 2 ? fast_sigmoid(w) : sigmoid_f(w));   // gelu_tanh(g) = g 0.5 (1 + tanh(w / 2)) = g sigmoid(w)
+      }
+      store_row<V>(out + (size_t)(s0 + j + q) * out_stride + c, o);
     }
   }
-  if (r0 + n == len) *slot = S;
+  if (r0 + n == len) store_row<V>(slot, S);
 }
 
 template <typename ST>
@@ -454,25 +504,37 @@ int launch_lru_conv(void* u, const void* proj_, long long stride, const float* x
   return check_cuda(cudaGetLastError(), "hyb_lru_conv");
 }
 
+template <typename ST, int V>
+int launch_lru_scan_cols(void* out, long long out_stride, float* state, float* sums, const void* u, const float* z, const void* proj, long long stride,
+                         const float* y_bias, const float* r_bias, const float* i_bias, const float* rate, const int* tile_entry, const int* tile_row0,
+                         int n_tiles, int n_short, const int* entry_start, const int* entry_len, const int* entry_slot, const int* entry_pos0, int T, int E,
+                         int W, int blocks, int tile_rows, int long_min, cudaStream_t s) {
+  const int cols = (W + 128 * V - 1) / (128 * V);
+  if (n_tiles > 0) {
+    dim3 grid(n_tiles, cols);
+    lru_tile_sums_kernel<ST, V><<<grid, 128, 0, s>>>(sums, (const ST*)u, z, r_bias, i_bias, rate, tile_entry, tile_row0, entry_start, entry_len, T, W, blocks,
+                                                     tile_rows);
+    lru_tile_starts_kernel<<<dim3(n_tiles, (W + 127) / 128), 128, 0, s>>>(sums, state, tile_entry, tile_row0, entry_len, entry_slot, entry_pos0, W, tile_rows);
+    lru_scan_kernel<ST, V><<<grid, 128, 0, s>>>((ST*)out, out_stride, state, sums, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias, rate,
+                                                tile_entry, tile_row0, entry_start, entry_len, entry_slot, entry_pos0, 1, long_min, T, W, blocks, tile_rows);
+  }
+  if (n_short > 0)
+    lru_scan_kernel<ST, V><<<dim3(E, cols), 128, 0, s>>>((ST*)out, out_stride, state, nullptr, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias,
+                                                         rate, nullptr, nullptr, entry_start, entry_len, entry_slot, entry_pos0, 0, long_min, T, W, blocks,
+                                                         tile_rows);
+  return check_cuda(cudaGetLastError(), "hyb_lru_scan");
+}
+
 template <typename ST>
 int launch_lru_scan(void* out, long long out_stride, float* state, float* sums, const void* u, const float* z, const void* proj, long long stride,
                     const float* y_bias, const float* r_bias, const float* i_bias, const float* rate, const int* tile_entry, const int* tile_row0,
                     int n_tiles, int n_short, const int* entry_start, const int* entry_len, const int* entry_slot, const int* entry_pos0, int T, int E,
                     int W, int blocks, int tile_rows, int long_min, cudaStream_t s) {
-  const int cols = (W + 127) / 128;
-  if (n_tiles > 0) {
-    dim3 grid(n_tiles, cols);
-    lru_tile_sums_kernel<ST><<<grid, 128, 0, s>>>(sums, (const ST*)u, z, r_bias, i_bias, rate, tile_entry, tile_row0, entry_start, entry_len, T, W, blocks,
-                                                  tile_rows);
-    lru_tile_starts_kernel<<<grid, 128, 0, s>>>(sums, state, tile_entry, tile_row0, entry_slot, entry_pos0, n_tiles, W);
-    lru_scan_kernel<ST><<<grid, 128, 0, s>>>((ST*)out, out_stride, state, sums, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias, rate,
-                                             tile_entry, tile_row0, entry_start, entry_len, entry_slot, entry_pos0, 1, long_min, T, W, blocks, tile_rows);
-  }
-  if (n_short > 0)
-    lru_scan_kernel<ST><<<dim3(E, cols), 128, 0, s>>>((ST*)out, out_stride, state, nullptr, (const ST*)u, z, (const ST*)proj, stride, y_bias, r_bias, i_bias,
-                                                      rate, nullptr, nullptr, entry_start, entry_len, entry_slot, entry_pos0, 0, long_min, T, W, blocks,
-                                                      tile_rows);
-  return check_cuda(cudaGetLastError(), "hyb_lru_scan");
+  // two channels per thread for prompts; a step of few rows needs the threads
+  const bool two = n_tiles > 0 && (W / blocks) % 2 == 0 && stride % 2 == 0 && out_stride % 2 == 0 && aligned(u, 8) && aligned(z, 8) && aligned(proj, 8) && aligned(out, 8);
+  auto run = two ? launch_lru_scan_cols<ST, 2> : launch_lru_scan_cols<ST, 1>;
+  return run(out, out_stride, state, sums, u, z, proj, stride, y_bias, r_bias, i_bias, rate, tile_entry, tile_row0, n_tiles, n_short, entry_start, entry_len,
+             entry_slot, entry_pos0, T, E, W, blocks, tile_rows, long_min, s);
 }
 
 }  // namespace
